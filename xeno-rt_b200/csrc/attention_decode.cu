@@ -34,6 +34,12 @@ __device__ __forceinline__ bool split_live(int split, int chunk, int first_key, 
   return split_begin(split, chunk, first_key) < len;
 }
 
+// A head's sink (a learned score without a key or a value): its term of the softmax's denominator in the base-2 domain of
+// the reference value m.  sinks: [n_heads] or null.
+__device__ __forceinline__ float sink_term(const float* sinks, int head, float m) {
+  return sinks != nullptr ? exp2f(sinks[head] * 1.4426950408889634f - m) : 0.f;
+}
+
 // What every form of the kernel does once its four warps have left their running state in the merge
 // area [warps][16 rows] of shared memory: merge them in warp order, write the output (one split) or
 // this split's partials, and, with counters, let the block that brings the last split merge all.
@@ -41,7 +47,7 @@ __device__ __forceinline__ void decode_finish(unsigned char* smem, __nv_bfloat16
                                               float* __restrict__ part_o, float* __restrict__ part_ml,
                                               int* __restrict__ counters, int tok, int kv_head, int split,
                                               int n_splits, int chunk, int first_key, int len, int group, int n_heads,
-                                              int n_kv_heads, int head_dim) {
+                                              int n_kv_heads, int head_dim, const float* __restrict__ sinks) {
   float* merge_m = reinterpret_cast<float*>(smem);                 // [warps][16]
   float* merge_l = merge_m + DEC_WARPS * 16;                       // [warps][16]
   float* merge_o = merge_l + DEC_WARPS * 16;                       // [warps][16][head_dim + 8]: rows in different banks
@@ -62,6 +68,7 @@ __device__ __forceinline__ void decode_finish(unsigned char* smem, __nv_bfloat16
     }
     const int head = kv_head * group + row;
     if (n_splits == 1) {
+      l += sink_term(sinks, head, m);
       out[((size_t)tok * n_heads + head) * head_dim + d] = __float2bfloat16_rn(o / l);
     } else {
       const size_t p = ((size_t)tok * n_heads + head) * n_splits + split;
@@ -109,7 +116,7 @@ __device__ __forceinline__ void decode_finish(unsigned char* smem, __nv_bfloat16
       all_m[row * n_splits + s] = f;
       l += f * all_l[row * n_splits + s];
     }
-    row_l[row] = l;
+    row_l[row] = l + sink_term(sinks, kv_head * group + row, m);
   }
   __syncthreads();
   for (int idx = threadIdx.x; idx < group * head_dim; idx += blockDim.x) {
@@ -136,8 +143,8 @@ attention_decode_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
                         const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pool,
                         const __nv_bfloat16* __restrict__ v_pool, const int* __restrict__ tok_slot,
                         const int* __restrict__ tok_pos, const int* __restrict__ block_table, int max_blocks,
-                        int n_heads, int n_kv_heads, int head_dim, float scale_log2, int window, int chunk,
-                        int n_splits, int* __restrict__ counters) {
+                        int n_heads, int n_kv_heads, int head_dim, float scale_log2, const KeyRange range, int chunk,
+                        int n_splits, int* __restrict__ counters, const float* __restrict__ sinks) {
   constexpr int D_TILES = HD_MAX / 8;
   extern __shared__ __align__(16) unsigned char smem[];
   pdl_trigger();
@@ -154,7 +161,7 @@ attention_decode_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
   }
   const int pos = tok_pos[tok];
   const int len = pos + 1;
-  const int first_key = window > 0 ? max(0, len - window) : 0;
+  const int first_key = range.first(len - 1);
   const int begin = split_begin(split, chunk, first_key);
   const int end = split_end(split, chunk, first_key, len);
   if (begin >= end) return;  // this split holds no visible key: the combine step skips it too
@@ -275,14 +282,15 @@ attention_decode_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
     }
   }
   decode_finish(smem, out, part_o, part_ml, counters, tok, kv_head, split, n_splits, chunk, first_key, len, group, n_heads,
-                n_kv_heads, head_dim);
+                n_kv_heads, head_dim, sinks);
 }
 
 // One warp per (token, head): merges the splits' partials in split order.
 __global__ void attention_combine_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ part_o,
                                          const float* __restrict__ part_ml, const int* __restrict__ tok_slot,
                                          const int* __restrict__ tok_pos, int n_tokens, int n_heads, int head_dim,
-                                         int window, int chunk, int n_splits) {
+                                         const KeyRange range, int chunk, int n_splits,
+                                         const float* __restrict__ sinks) {
   pdl_trigger();
   pdl_wait();
   const int warp_global = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
@@ -294,7 +302,7 @@ __global__ void attention_combine_kernel(__nv_bfloat16* __restrict__ out, const 
     return;
   }
   const int len = tok_pos[tok] + 1;
-  const int first_key = window > 0 ? max(0, len - window) : 0;
+  const int first_key = range.first(len - 1);
   const size_t base = (size_t)warp_global * n_splits;
   float m = -INFINITY;
   for (int s = 0; s < n_splits; ++s) {
@@ -321,6 +329,7 @@ __global__ void attention_combine_kernel(__nv_bfloat16* __restrict__ out, const 
       acc[j] += f * o;
     }
   }
+  l += sink_term(sinks, warp_global - tok * n_heads, m);
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
     const int d = lane + 32 * j;
@@ -397,9 +406,9 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                             __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
                             const __nv_bfloat16* __restrict__ q, const int* __restrict__ tok_slot,
                             const int* __restrict__ tok_pos, const int* __restrict__ block_table, int max_blocks,
-                            int n_heads, int n_kv_heads, int head_dim, float scale_log2, int window, int chunk,
+                            int n_heads, int n_kv_heads, int head_dim, float scale_log2, const KeyRange range, int chunk,
                             int n_splits, int* __restrict__ counters, int* __restrict__ error_flag, int clustered,
-                            int stages, const DecodeFusedInput fused) {
+                            int stages, const DecodeFusedInput fused, const float* __restrict__ sinks) {
   constexpr int D_TILES = HD_MAX / 8;
   __shared__ __align__(16) __nv_bfloat16 newest[2][HD_MAX];  // the step's own key and value of this kv head
   extern __shared__ unsigned char smem_raw[];
@@ -422,7 +431,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     return;
   }
   const int len = tok_pos[tok] + 1;
-  const int first_key = window > 0 ? max(0, len - window) : 0;
+  const int first_key = range.first(len - 1);
   const int begin = split_begin(split, chunk, first_key);
   const int end = split_end(split, chunk, first_key, len);
   const bool has_keys = begin < end;
@@ -478,7 +487,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   // before this one writes that key; when this kernel writes it itself, the tile's row is patched below.
   const bool holds_newest = has_keys && len - 1 >= begin && len - 1 < end;
   const bool writes_newest = fused.qkv != nullptr && fused.k_pool != nullptr && holds_newest;
-  const bool early = has_keys && (fused.qkv != nullptr || begin + XRT_BLOCK_TOKENS <= len - 1);
+  // (A layer that reads another layer's cache has a newest key that a kernel of this step wrote.)
+  const bool early = has_keys && ((fused.qkv != nullptr && fused.k_pool != nullptr) || begin + XRT_BLOCK_TOKENS <= len - 1);
   if (asks && early) issue_tile(0, 0, block_of(0));
   pdl_wait();
   uint32_t qb[D_TILES / 2][2];
@@ -660,7 +670,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   }
   if (!clustered) {
     decode_finish(smem, out, part_o, part_ml, counters, tok, kv_head, split, n_splits, chunk, first_key, len, group, n_heads,
-                  n_kv_heads, head_dim);
+                  n_kv_heads, head_dim, sinks);
     return;
   }
 
@@ -717,6 +727,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         l += f * ls[s2];
         o += f * os[s2];
       }
+      l += sink_term(sinks, kv_head * group + row, m);
       out[((size_t)tok * n_heads + (size_t)kv_head * group) * head_dim + idx] = __float2bfloat16_rn(o / l);
     }
   }
@@ -778,8 +789,8 @@ template <int HD_MAX>
 int launch_decode_tma(__nv_bfloat16* out, float* part_o, float* part_ml, const __nv_bfloat16* q,
                       const __nv_bfloat16* k_pool, const __nv_bfloat16* v_pool, long long pool_rows, const int* tok_slot,
                       const int* tok_pos, const int* block_table, int max_blocks, int n_tokens, int n_heads, int n_kv_heads,
-                      int head_dim, float scale, int window, int chunk, int n_splits, int* counters, int* error_flag,
-                      cudaStream_t stream, bool* merged, const DecodeFusedInput& fused, bool clusters) {
+                      int head_dim, float scale, const KeyRange& range, int chunk, int n_splits, int* counters, int* error_flag,
+                      cudaStream_t stream, bool* merged, const DecodeFusedInput& fused, bool clusters, const float* sinks) {
   CUtensorMap map_k, map_v;
   if (!dec_make_map(&map_k, k_pool, pool_rows, head_dim) || !dec_make_map(&map_v, v_pool, pool_rows, head_dim))
     return XRT_ERR_UNSUPPORTED;
@@ -852,8 +863,8 @@ int launch_decode_tma(__nv_bfloat16* out, float* part_o, float* part_ml, const _
   config.attrs = n_attrs ? attrs : nullptr;
   config.numAttrs = n_attrs;
   cudaLaunchKernelEx(&config, kernel, map_k, map_v, out, part_o, part_ml, q, tok_slot, tok_pos, block_table, max_blocks,
-                     n_heads, n_kv_heads, head_dim, scale * 1.4426950408889634f, window, chunk, n_splits, counters, error_flag,
-                     clustered ? 1 : 0, stages, fused);
+                     n_heads, n_kv_heads, head_dim, scale * 1.4426950408889634f, range, chunk, n_splits, counters, error_flag,
+                     clustered ? 1 : 0, stages, fused, sinks);
   return launch_status();
 }
 
@@ -861,7 +872,8 @@ template <int HD_MAX, bool BY_HEADS>
 int launch_decode_as(__nv_bfloat16* out, float* part_o, float* part_ml, const __nv_bfloat16* q,
                   const __nv_bfloat16* k_pool, const __nv_bfloat16* v_pool, const int* tok_slot, const int* tok_pos,
                   const int* block_table, int max_blocks, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
-                  float scale, int window, int chunk, int n_splits, int* counters, cudaStream_t stream) {
+                  float scale, const KeyRange& range, int chunk, int n_splits, int* counters, cudaStream_t stream,
+                  const float* sinks) {
   const int tile_bytes = XRT_BLOCK_TOKENS * (head_dim * 2 + 16);
   const int merge_bytes = DEC_WARPS * 16 * (2 + head_dim + 8) * (int)sizeof(float);
   const int smem = max(4 * tile_bytes, merge_bytes);
@@ -875,7 +887,7 @@ int launch_decode_as(__nv_bfloat16* out, float* part_o, float* part_ml, const __
   dim3 grid(n_splits, n_kv_heads, n_tokens);
   launch_kernel(kernel, grid, dim3(DEC_WARPS * 32), (size_t)smem, stream, out, part_o, part_ml, q, k_pool, v_pool,
                 tok_slot, tok_pos, block_table, max_blocks, n_heads, n_kv_heads, head_dim,
-                scale * 1.4426950408889634f, window, chunk, n_splits, counters);
+                scale * 1.4426950408889634f, range, chunk, n_splits, counters, sinks);
   return launch_status();
 }
 
@@ -887,8 +899,8 @@ template <int HD_MAX>
 int launch_decode(__nv_bfloat16* out, float* part_o, float* part_ml, const __nv_bfloat16* q,
                   const __nv_bfloat16* k_pool, const __nv_bfloat16* v_pool, long long pool_rows, const int* tok_slot,
                   const int* tok_pos, const int* block_table, int max_blocks, int n_tokens, int n_heads, int n_kv_heads,
-                  int head_dim, float scale, int window, int chunk, int n_splits, int* counters, int* error_flag,
-                  cudaStream_t stream, bool* merged, const DecodeFusedInput& fused, bool clusters) {
+                  int head_dim, float scale, const KeyRange& range, int chunk, int n_splits, int* counters, int* error_flag,
+                  cudaStream_t stream, bool* merged, const DecodeFusedInput& fused, bool clusters, const float* sinks) {
   *merged = false;
   const bool rows_only = tuning().decode_attention == 1, copies_only = tuning().decode_attention == 2;
   if (n_heads / n_kv_heads <= 8 && !rows_only && !copies_only && pool_rows > 0 && head_dim % 64 == 0 &&
@@ -898,17 +910,17 @@ int launch_decode(__nv_bfloat16* out, float* part_o, float* part_ml, const __nv_
                                  fused.v_offset % 4 != 0 || (((uintptr_t)fused.qkv | (uintptr_t)fused.cos_sin) & 15) != 0))
       return XRT_ERR_UNSUPPORTED;
     return launch_decode_tma<HD_MAX>(out, part_o, part_ml, q, k_pool, v_pool, pool_rows, tok_slot, tok_pos, block_table,
-                                     max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, window, chunk, n_splits,
-                                     counters, error_flag, stream, merged, fused, clusters);
+                                     max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, range, chunk, n_splits,
+                                     counters, error_flag, stream, merged, fused, clusters, sinks);
   }
   if (fused.qkv != nullptr) return XRT_ERR_UNSUPPORTED;  // only the kernel above rotates and writes the cache itself
   if (n_heads / n_kv_heads <= 8 && !rows_only)
     return launch_decode_as<HD_MAX, true>(out, part_o, part_ml, q, k_pool, v_pool, tok_slot, tok_pos, block_table,
-                                          max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, window, chunk,
-                                          n_splits, counters, stream);
+                                          max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, range, chunk,
+                                          n_splits, counters, stream, sinks);
   return launch_decode_as<HD_MAX, false>(out, part_o, part_ml, q, k_pool, v_pool, tok_slot, tok_pos, block_table,
-                                         max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, window, chunk,
-                                         n_splits, counters, stream);
+                                         max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, range, chunk,
+                                         n_splits, counters, stream, sinks);
 }
 
 // The merge by a (token, kv head)'s last block keeps group * (2 * n_splits + 1) floats in the block's
@@ -938,9 +950,10 @@ namespace xrt {
 static int attention_decode_impl(void* out, float* part_o, float* part_ml, const void* q, const void* k_pool,
                                  const void* v_pool, int n_blocks, const int* tok_slot, const int* tok_pos,
                                  const int* block_table, int max_blocks, int n_tokens, int n_heads, int n_kv_heads,
-                                 int head_dim, float scale, int window, int chunk, int n_splits, int* counters,
+                                 int head_dim, float scale, const KeyRange& range, int chunk, int n_splits, int* counters,
                                  int* error_flag, cudaStream_t stream, int* merged_out = nullptr,
-                                 const DecodeFusedInput& fused = DecodeFusedInput(), bool clusters = true) {
+                                 const DecodeFusedInput& fused = DecodeFusedInput(), bool clusters = true,
+                                 const float* sinks = nullptr) {
   if (n_tokens < 0 || n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || chunk <= 0 || n_splits <= 0)
     return XRT_ERR_ARGUMENT;
   if (head_dim % 16 != 0 || head_dim < 16 || head_dim > 256 || n_heads / n_kv_heads > 16 ||
@@ -958,8 +971,8 @@ static int attention_decode_impl(void* out, float* part_o, float* part_ml, const
   bool merged = false;  // the attention kernel merged its splits itself (as clusters)
   const long long pool_rows = (long long)n_blocks * n_kv_heads * XRT_BLOCK_TOKENS;  // 0: the pools' size is not known
 #define XRT_DECODE(HD) status = launch_decode<HD>(o, part_o, part_ml, qp, kp, vp, pool_rows, tok_slot, tok_pos, block_table, \
-                                                  max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, window,      \
-                                                  chunk, n_splits, counters, error_flag, stream, &merged, fused, clusters)
+                                                  max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, range,       \
+                                                  chunk, n_splits, counters, error_flag, stream, &merged, fused, clusters, sinks)
   if (head_dim <= 32) XRT_DECODE(32);
   else if (head_dim <= 64) XRT_DECODE(64);
   else if (head_dim <= 128) XRT_DECODE(128);
@@ -971,8 +984,8 @@ static int attention_decode_impl(void* out, float* part_o, float* part_ml, const
     const int warps = n_tokens * n_heads;
     const int threads = warps <= 1024 ? 64 : 256;  // few rows: two warps a block, so that they spread over the multiprocessors
     launch_kernel(attention_combine_kernel, dim3((warps * 32 + threads - 1) / threads), dim3(threads), 0, stream, o,
-                  (const float*)part_o, (const float*)part_ml, tok_slot, tok_pos, n_tokens, n_heads, head_dim, window,
-                  chunk, n_splits);
+                  (const float*)part_o, (const float*)part_ml, tok_slot, tok_pos, n_tokens, n_heads, head_dim, range,
+                  chunk, n_splits, sinks);
     return launch_status();
   }
   return XRT_OK;
@@ -997,10 +1010,11 @@ XRT_EXPORT int xrt_attention_decode(void* out, float* part_o, float* part_ml, co
                                     const void* v_pool, int n_blocks, const int* tok_slot, const int* tok_pos,
                                     const int* block_table, int max_blocks, int n_tokens, int n_heads, int n_kv_heads,
                                     int head_dim, float scale, int window, int chunk, int n_splits, int* error_flag,
-                                    cudaStream_t stream, int* merged, int clusters) {
+                                    cudaStream_t stream, int* merged, int clusters, const float* sinks,
+                                    int mask_chunk) {
   return xrt::attention_decode_impl(out, part_o, part_ml, q, k_pool, v_pool, n_blocks, tok_slot, tok_pos, block_table,
-                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, window, chunk, n_splits,
-                                    nullptr, error_flag, stream, merged, xrt::DecodeFusedInput(), clusters != 0);
+                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, xrt::key_range(window, mask_chunk), chunk, n_splits,
+                                    nullptr, error_flag, stream, merged, xrt::DecodeFusedInput(), clusters != 0, sinks);
 }
 
 // The same, with the merge done by the block that brings a (token, kv head)'s last split: one
@@ -1010,11 +1024,12 @@ XRT_EXPORT int xrt_attention_decode_fused(void* out, float* part_o, float* part_
                                           const void* k_pool, const void* v_pool, int n_blocks, const int* tok_slot,
                                           const int* tok_pos, const int* block_table, int max_blocks, int n_tokens,
                                           int n_heads, int n_kv_heads, int head_dim, float scale, int window, int chunk,
-                                          int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters) {
+                                          int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters, const float* sinks,
+                                    int mask_chunk) {
   if (counters == nullptr) return XRT_ERR_ARGUMENT;
   return xrt::attention_decode_impl(out, part_o, part_ml, q, k_pool, v_pool, n_blocks, tok_slot, tok_pos, block_table,
-                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, window, chunk, n_splits,
-                                    counters, error_flag, stream, merged, xrt::DecodeFusedInput(), clusters != 0);
+                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, xrt::key_range(window, mask_chunk), chunk, n_splits,
+                                    counters, error_flag, stream, merged, xrt::DecodeFusedInput(), clusters != 0, sinks);
 }
 
 // The same, fed with the 32-bit output of the q/k/v product instead of a rotated q: the kernel applies
@@ -1030,7 +1045,8 @@ XRT_EXPORT int xrt_attention_decode_qkv(void* out, float* part_o, float* part_ml
                                         int write_kv, void* k_pool, void* v_pool, int n_blocks, const int* tok_slot,
                                         const int* tok_pos, const int* block_table, int max_blocks, int n_tokens,
                                         int n_heads, int n_kv_heads, int head_dim, float scale, int window, int chunk,
-                                        int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters) {
+                                        int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters, const float* sinks,
+                                    int mask_chunk) {
   if (qkv == nullptr || (q_norm_w == nullptr) != (k_norm_w == nullptr) || n_blocks <= 0) return XRT_ERR_ARGUMENT;
   if (norm_dtype != XRT_F32 && norm_dtype != XRT_BF16) return XRT_ERR_UNSUPPORTED;
   xrt::DecodeFusedInput fused;
@@ -1041,8 +1057,8 @@ XRT_EXPORT int xrt_attention_decode_qkv(void* out, float* part_o, float* part_ml
   fused.k_pool = write_kv ? (__nv_bfloat16*)k_pool : nullptr;
   fused.v_pool = write_kv ? (__nv_bfloat16*)v_pool : nullptr;
   return xrt::attention_decode_impl(out, part_o, part_ml, nullptr, k_pool, v_pool, n_blocks, tok_slot, tok_pos, block_table,
-                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, window, chunk, n_splits,
-                                    counters, error_flag, stream, merged, fused, clusters != 0);
+                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, xrt::key_range(window, mask_chunk), chunk, n_splits,
+                                    counters, error_flag, stream, merged, fused, clusters != 0, sinks);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -1119,7 +1135,7 @@ int xrt_attention_decode_static(void* out, const void* q, const void* k_pool, co
   // the pools' size is not among this entry's arguments: 0 keeps it on the kernels that need no tensor map
   const int status = xrt_attention_decode(out, scratch + ml_floats, scratch, q, k_pool, v_pool, 0, tok_slot, tok_pos,
                                           block_table, max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale,
-                                          window, chunk, n_splits, nullptr, stream, nullptr, 1);
+                                          window, chunk, n_splits, nullptr, stream, nullptr, 1, nullptr, 0);
   if (status == XRT_ERR_ARGUMENT) xrt::refuse(message, message_len, "xrt_attention_decode_static: the kernel refused its arguments");
   if (status == XRT_ERR_UNSUPPORTED)
     xrt::refuse(message, message_len, "xrt_attention_decode_static: head_dim must be a multiple of 16 up to 256, at most "

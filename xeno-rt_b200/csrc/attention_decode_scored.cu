@@ -19,7 +19,8 @@ struct DecodeScoredArgs {
   float* partial;                // [tokens, heads, splits, head_dim + 2] (o, then m, l), or null with one split
   const __nv_bfloat16 *q, *k_pool, *v_pool;
   const int *tok_slot, *tok_pos, *block_table;
-  int max_blocks, n_heads, n_kv_heads, head_dim, window, chunk, n_splits;
+  int max_blocks, n_heads, n_kv_heads, head_dim, chunk, n_splits;
+  KeyRange range;
   float scale;
   ScoreOptions opt;
 };
@@ -42,7 +43,7 @@ __global__ void __launch_bounds__(DS_WARPS * 32) attention_decode_scored_kernel(
     return;
   }
   const int pos = a.tok_pos[t];
-  const int first = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int first = a.range.first(pos);
   const int kept = min(a.opt.keep_first, first);
   const int total = kept + pos - first + 1;
   const int v_begin = split * a.chunk, v_end = min(total, v_begin + a.chunk);
@@ -163,7 +164,7 @@ __global__ void __launch_bounds__(DS_WARPS * 32) attention_decode_scored_kernel(
       }
       const int head = kv * group + h0 + g;
       if (a.partial == nullptr) {
-        if (a.opt.sink) sum += expf(a.opt.sink_score - top);
+        if (a.opt.sink) sum += expf(sink_of(a.opt, head) - top);
         a.out[((size_t)t * a.n_heads + head) * hd + d] = __float2bfloat16_rn(o / sum);
       } else {
         float* dst = a.partial + (((size_t)t * a.n_heads + head) * a.n_splits + split) * (hd + 2);
@@ -177,7 +178,7 @@ __global__ void __launch_bounds__(DS_WARPS * 32) attention_decode_scored_kernel(
 // The splits of a (token, head), in index order.
 __global__ void attention_decode_scored_merge_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ partial,
                                                      const int* __restrict__ tok_slot, int n_heads, int head_dim,
-                                                     int n_splits, int sink, float sink_score) {
+                                                     int n_splits, const ScoreOptions opt) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x, head = blockIdx.y;
@@ -193,7 +194,7 @@ __global__ void attention_decode_scored_merge_kernel(__nv_bfloat16* __restrict__
       sum = fmaf(p[head_dim + 1], f, sum);
       o = fmaf(p[d], f, o);
     }
-    if (sink) sum += expf(sink_score - top);
+    if (opt.sink) sum += expf(sink_of(opt, head) - top);
     out[((size_t)t * n_heads + head) * head_dim + d] = __float2bfloat16_rn(o / sum);
   }
 }
@@ -220,7 +221,7 @@ XRT_EXPORT int xrt_attention_decode_scored(void* out, float* partial, const void
                                            const int* tok_slot, const int* tok_pos, const int* block_table, int max_blocks,
                                            int n_tokens, int n_heads, int n_kv_heads, int head_dim, float scale, int window,
                                            int keep_first, float softcap, float distance_rate, int sink, float sink_score,
-                                           int chunk, int n_splits, cudaStream_t stream) {
+                                           const float* sinks, int mask_chunk, int chunk, int n_splits, cudaStream_t stream) {
   if (n_tokens < 0 || n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads || head_dim <= 0 || chunk <= 0 || n_splits <= 0)
     return XRT_ERR_ARGUMENT;
   if (head_dim % 8 || head_dim > 256 || chunk % 32 || n_tokens > 65535 * 32 || n_kv_heads > 65535 || n_splits > 65535 ||
@@ -234,12 +235,13 @@ XRT_EXPORT int xrt_attention_decode_scored(void* out, float* partial, const void
   a.q = (const __nv_bfloat16*)q; a.k_pool = (const __nv_bfloat16*)k_pool; a.v_pool = (const __nv_bfloat16*)v_pool;
   a.tok_slot = tok_slot; a.tok_pos = tok_pos; a.block_table = block_table;
   a.max_blocks = max_blocks; a.n_heads = n_heads; a.n_kv_heads = n_kv_heads; a.head_dim = head_dim;
-  a.window = window; a.chunk = chunk; a.n_splits = n_splits; a.scale = scale;
+  a.range = xrt::key_range(window, mask_chunk); a.chunk = chunk; a.n_splits = n_splits; a.scale = scale;
   a.opt.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
   a.opt.softcap = softcap;
   a.opt.distance_rate = distance_rate;
   a.opt.sink = sink;
   a.opt.sink_score = sink_score;
+  a.opt.sinks = sinks;
   const int group = n_heads / n_kv_heads;
   const int pairs = head_dim <= 64 ? 1 : (head_dim <= 128 ? 2 : 4);
   int status;
@@ -254,6 +256,6 @@ XRT_EXPORT int xrt_attention_decode_scored(void* out, float* partial, const void
 #undef XRT_DS
   if (status != XRT_OK || n_splits == 1) return status;
   xrt::launch_kernel(xrt::attention_decode_scored_merge_kernel, dim3(n_tokens, n_heads), dim3(head_dim >= 128 ? 128 : 64), 0,
-                     stream, (__nv_bfloat16*)out, (const float*)partial, tok_slot, n_heads, head_dim, n_splits, sink, sink_score);
+                     stream, (__nv_bfloat16*)out, (const float*)partial, tok_slot, n_heads, head_dim, n_splits, a.opt);
   return xrt::launch_status();
 }

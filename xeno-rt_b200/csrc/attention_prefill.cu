@@ -26,7 +26,7 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
                          const __nv_bfloat16* __restrict__ k_pool, const __nv_bfloat16* __restrict__ v_pool,
                          const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
                          const int* __restrict__ seq_start, const int* __restrict__ block_table, int max_blocks,
-                         int n_heads, int n_kv_heads, int head_dim, float scale_log2, int window,
+                         int n_heads, int n_kv_heads, int head_dim, float scale_log2, const KeyRange range,
                          const ScoreOptions opt) {
   constexpr int D_TILES = HD_MAX / 8;
   extern __shared__ __align__(16) unsigned char smem[];
@@ -54,7 +54,7 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
   for (int r = 0; r < 2; ++r) {
     const int pos = start + rows[r];
     key_hi[r] = rows[r] < n_new ? pos + 1 : 0;  // a row beyond the sequence sees nothing
-    key_lo[r] = window > 0 ? max(0, pos + 1 - window) : 0;
+    key_lo[r] = range.first(pos);
   }
   uint32_t qf[D_TILES / 2][4];
 #pragma unroll
@@ -70,7 +70,7 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
   // keys the block needs: from the first row's window edge to the last row's position
   const int last_row = min(row0 + PRE_ROWS, n_new) - 1;
   const int block_hi = start + last_row + 1;                                        // exclusive
-  const int block_lo = window > 0 ? max(0, start + row0 + 1 - window) : 0;
+  const int block_lo = range.first(start + row0);
   const int first_tile = block_lo / XRT_BLOCK_TOKENS;
   // tiles of keys that stay visible behind the window come first; a tile is walked once
   const int keep_tiles = SCORED ? min((opt.keep_first + XRT_BLOCK_TOKENS - 1) / XRT_BLOCK_TOKENS, first_tile) : 0;
@@ -86,10 +86,10 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
   const int warp_first_row = row0 + warp * 16;
   const int warp_last_row = min(warp_first_row + 15, n_new - 1);
   const int warp_hi = warp_first_row < n_new ? start + warp_last_row + 1 : 0;
-  const int warp_lo = window > 0 ? max(0, start + warp_first_row + 1 - window) : 0;
+  const int warp_lo = range.first(start + warp_first_row);
   // every row of the warp sees the keys in [warp_max_lo, warp_min_hi): a tile inside needs no mask
   const int warp_min_hi = warp_first_row < n_new ? start + warp_first_row + 1 : 0;
-  const int warp_max_lo = window > 0 ? max(0, start + warp_last_row + 1 - window) : 0;
+  const int warp_max_lo = range.first(start + max(warp_last_row, 0));
   const bool partial_warp = warp_first_row + 15 >= n_new;  // some rows lie beyond the sequence and see nothing
 
   const int* blocks = block_table + (size_t)slot * max_blocks;
@@ -129,7 +129,7 @@ attention_prefill_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* _
     st.l[r] += __shfl_xor_sync(0xffffffffu, st.l[r], 1);
     st.l[r] += __shfl_xor_sync(0xffffffffu, st.l[r], 2);
     // a sink: one more term of the denominator, exp(sink_score), in the base-2 domain of the running maximum
-    if (opt.sink && st.m[r] != -INFINITY) st.l[r] += exp2f(opt.sink_score * 1.4426950408889634f - st.m[r]);
+    if (opt.sink && st.m[r] != -INFINITY) st.l[r] += exp2f(sink_of(opt, head) * 1.4426950408889634f - st.m[r]);
   }
 #pragma unroll
   for (int dt = 0; dt < D_TILES; ++dt) {
@@ -150,7 +150,7 @@ template <int HD_MAX, bool SCORED>
 int launch_prefill_of(__nv_bfloat16* out, const __nv_bfloat16* q, const __nv_bfloat16* k_pool, const __nv_bfloat16* v_pool,
                    const int* cu_seqlens, const int* seq_slot, const int* seq_start, const int* block_table,
                    int max_blocks, int n_seqs, int max_new, int n_heads, int n_kv_heads, int head_dim, float scale,
-                   int window, const ScoreOptions& opt, cudaStream_t stream) {
+                   const KeyRange& range, const ScoreOptions& opt, cudaStream_t stream) {
   const int smem = 4 * XRT_BLOCK_TOKENS * (head_dim * 2 + 16);
   auto kernel = attention_prefill_kernel<HD_MAX, SCORED>;
   static int smem_allowed = 0;
@@ -162,7 +162,7 @@ int launch_prefill_of(__nv_bfloat16* out, const __nv_bfloat16* q, const __nv_bfl
   dim3 grid(n_heads, n_seqs, (max_new + PRE_ROWS - 1) / PRE_ROWS);
   kernel<<<grid, PRE_WARPS * 32, smem, stream>>>(out, q, k_pool, v_pool, cu_seqlens, seq_slot, seq_start, block_table,
                                                 max_blocks, n_heads, n_kv_heads, head_dim,
-                                                SCORED ? scale : scale * 1.4426950408889634f, window, opt);
+                                                SCORED ? scale : scale * 1.4426950408889634f, range, opt);
   return launch_status();
 }
 
@@ -170,12 +170,12 @@ template <int HD_MAX>
 int launch_prefill(__nv_bfloat16* out, const __nv_bfloat16* q, const __nv_bfloat16* k_pool, const __nv_bfloat16* v_pool,
                    const int* cu_seqlens, const int* seq_slot, const int* seq_start, const int* block_table,
                    int max_blocks, int n_seqs, int max_new, int n_heads, int n_kv_heads, int head_dim, float scale,
-                   int window, const ScoreOptions& opt, cudaStream_t stream) {
+                   const KeyRange& range, const ScoreOptions& opt, cudaStream_t stream) {
   if (opt.keep_first > 0 || opt.softcap > 0.f || opt.distance_rate > 0.f)
     return launch_prefill_of<HD_MAX, true>(out, q, k_pool, v_pool, cu_seqlens, seq_slot, seq_start, block_table, max_blocks,
-                                           n_seqs, max_new, n_heads, n_kv_heads, head_dim, scale, window, opt, stream);
+                                           n_seqs, max_new, n_heads, n_kv_heads, head_dim, scale, range, opt, stream);
   return launch_prefill_of<HD_MAX, false>(out, q, k_pool, v_pool, cu_seqlens, seq_slot, seq_start, block_table, max_blocks,
-                                          n_seqs, max_new, n_heads, n_kv_heads, head_dim, scale, window, opt, stream);
+                                          n_seqs, max_new, n_heads, n_kv_heads, head_dim, scale, range, opt, stream);
 }
 
 }  // namespace xrt
@@ -189,13 +189,15 @@ XRT_EXPORT int xrt_attention_prefill(void* out, const void* q, const void* k_poo
                                      const int* block_table, int max_blocks, int n_seqs, int max_new, int n_heads,
                                      int n_kv_heads, int head_dim, float scale, int window, int keep_first,
                                      float softcap, float distance_rate, int sink, float sink_score,
-                                     cudaStream_t stream) {
+                                     const float* sinks, int mask_chunk, cudaStream_t stream) {
   xrt::ScoreOptions opt;
   opt.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
   opt.softcap = softcap;
   opt.distance_rate = distance_rate;
   opt.sink = sink;
   opt.sink_score = sink_score;
+  opt.sinks = sinks;
+  const xrt::KeyRange range = xrt::key_range(window, mask_chunk);
   if (n_seqs < 0 || max_new < 0 || n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return XRT_ERR_ARGUMENT;
   if (head_dim % 16 != 0 || head_dim < 16 || head_dim > 256 || n_seqs > 65535 || (max_new + xrt::PRE_ROWS - 1) / xrt::PRE_ROWS > 65535) return XRT_ERR_UNSUPPORTED;
   if (n_seqs == 0 || max_new == 0) return XRT_OK;
@@ -205,7 +207,7 @@ XRT_EXPORT int xrt_attention_prefill(void* out, const void* q, const void* k_poo
   auto* vp = (const __nv_bfloat16*)v_pool;
 #define XRT_PREFILL(HD) return xrt::launch_prefill<HD>(o, qp, kp, vp, cu_seqlens, seq_slot, seq_start, block_table, \
                                                        max_blocks, n_seqs, max_new, n_heads, n_kv_heads, head_dim,  \
-                                                       scale, window, opt, stream)
+                                                       scale, range, opt, stream)
   if (head_dim <= 32) XRT_PREFILL(32);
   if (head_dim <= 64) XRT_PREFILL(64);
   if (head_dim <= 128) XRT_PREFILL(128);

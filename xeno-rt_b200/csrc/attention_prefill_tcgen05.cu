@@ -3,7 +3,9 @@
 // 0 .. start + t, read from the cache so that earlier context is included.)
 //
 // A block owns 128 consecutive new tokens of one sequence for one query head and walks the
-// sequence's keys in steps of 128 (two cache blocks of 64).  Six warps:
+// sequence's keys in steps of 128 (two cache blocks of 64) from the cache block of the first row's first visible key
+// (KeyRange in common.cuh: all keys, a window, or the query's own chunk of positions).  A head may have a sink: one
+// more term of the softmax's denominator, added to the row's sum at the end.  Six warps:
 //   warp 0    TMA: the Q tile once, then for each step its K and V tiles ([128 keys x 128], as boxes
 //             of 64 keys x 64 dims, 128-byte swizzle) into a ring of three stages.  K and V of a stage
 //             have barriers of their own: K is free again after the step's QK^T, a whole step before V.
@@ -59,7 +61,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                                  const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
                                  const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
                                  const int* __restrict__ seq_start, const int* __restrict__ block_table, int max_blocks,
-                                 int n_heads, int n_kv_heads, float scale_log2, int* __restrict__ error_flag) {
+                                 int n_heads, int n_kv_heads, float scale_log2, int* __restrict__ error_flag,
+                                 const KeyRange range, const float* __restrict__ sinks) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   unsigned char* q_tiles = smem;                                   // [NH] x 32 KB
@@ -93,7 +96,10 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
   const int start = seq_start[seq];
   const int kv_head = head0 / (n_heads / n_kv_heads);  // the same for all NH heads: NH divides the group
   const int last_row = min(row0 + FA_ROWS, n_new) - 1;
-  const int n_tiles = (start + last_row + 1 + FA_KEYS - 1) / FA_KEYS;  // keys 0 .. position of the last row
+  // keys from the cache block of the first row's first visible key to the last row's position
+  const int first_block = range.first(start + row0) / XRT_BLOCK_TOKENS;
+  const int key_base = first_block * XRT_BLOCK_TOKENS;
+  const int n_tiles = (start + last_row + 1 - key_base + FA_KEYS - 1) / FA_KEYS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   static_assert(NH * (2 * FA_KEYS + FA_HD + FA_P_BUFFERS * FA_P_COLS) <= 512, "S buffers, O and P buffers must fit in TMEM");
   constexpr int TMEM_COLS = 512;  // S: NH x 2 buffers x 128 columns; O: NH x 128; P: NH x 2 buffers x 64
@@ -152,7 +158,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         int pool_row[2];  // the step's two cache blocks; beyond the last one the last again (masked)
 #pragma unroll
         for (int part = 0; part < 2; ++part)
-          pool_row[part] = (blocks[min(2 * j + part, n_blocks - 1)] * n_kv_heads + kv_head) * XRT_BLOCK_TOKENS;
+          pool_row[part] = (blocks[min(first_block + 2 * j + part, n_blocks - 1)] * n_kv_heads + kv_head) * XRT_BLOCK_TOKENS;
         ok = mbar_wait(smem_u32(&k_empty[s]), ((j / FA_STAGES) & 1) ^ 1, abort_flag);
         if (!ok) break;
         mbar_arrive_expect_tx(smem_u32(&k_full[s]), 2 * FA_KV_HALF);
@@ -230,7 +236,9 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     const int r = quarter * 32 + lane;           // row of the tile = TMEM lane
     const int row = row0 + r;                    // new-token index in the sequence
     const bool row_live = row < n_new;
-    const int key_hi = row_live ? start + row + 1 : 0;  // keys [0, key_hi) are visible
+    const int key_hi = row_live ? start + row + 1 : 0;  // keys [key_lo, key_hi) are visible
+    const int key_lo = range.first(start + row);
+    const int all_lo = range.first(start + last_row);   // from here on no row's range has yet to begin
     const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
     const uint32_t my_s = tmem_s + lane_base + h * 2 * FA_KEYS, my_o = tmem_o + lane_base + h * FA_HD;
     float m_ref = -INFINITY, l_run = 0.f;  // the reference value of the exponents (scaled, base 2) and the sum
@@ -258,9 +266,13 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
       fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&s_empty[b]));  // the tensor core may write the block after next into this buffer
-      const int key0 = j * FA_KEYS;
-      // Only blocks that reach past the first row's last visible key can hide a key from a row
-      // (uniform over the thread block); every other block skips the comparisons.
+      const int key0 = key_base + j * FA_KEYS;
+      // Only blocks that reach past the first row's last visible key, or begin before the last row's first one, can
+      // hide a key from a row (uniform over the thread block); every other block skips the comparisons.
+      if (key0 < all_lo) {
+#pragma unroll
+        for (int i = 0; i < FA_KEYS; ++i) s[i] = (key0 + i >= key_lo) ? s[i] : -INFINITY;
+      }
       if (key0 + FA_KEYS > start + row0 + 1) {
 #pragma unroll
         for (int i = 0; i < FA_KEYS; ++i) s[i] = (key0 + i < key_hi) ? s[i] : -INFINITY;
@@ -330,6 +342,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     if (ok && n_tiles > 0) ok = mbar_wait(smem_u32(pv_done), (uint32_t)(n_tiles - 1) & 1u, abort_flag);
     if (ok && n_tiles > 0) {
       fence_after();
+      if (sinks != nullptr) l_run += exp2f(sinks[head] * 1.4426950408889634f - m_ref);
       const float inv = row_live ? 1.0f / l_run : 0.f;
       __nv_bfloat16* dst = out + ((size_t)(tok0 + row) * n_heads + head) * FA_HD;
 #pragma unroll
@@ -373,13 +386,15 @@ static bool fa_make_map(CUtensorMap* map, const void* base, long long rows, int 
 
 // q, out: bfloat16 [n_tokens, n_heads * 128], the sequences' new tokens end to end (cu_seqlens[n_seqs + 1]);
 // pools: bfloat16 [n_blocks, n_kv_heads, 64, 128]; seq_slot[n_seqs] (< 0: skipped), seq_start[n_seqs] = tokens each
-// sequence held before this step; max_new = the most new tokens any sequence brings.  Head size 128 only, no window.
+// sequence held before this step; max_new = the most new tokens any sequence brings.  Head size 128 only.  `window` and `mask_chunk` bound
+// the keys a query sees (KeyRange; 0 = no bound); sinks: float32 [n_heads] or null.
 // error_flag (may be null) is set to 5 if a bounded wait ran out.
 XRT_EXPORT int xrt_attention_prefill_tcgen05(void* out, const void* q, const void* k_pool, const void* v_pool,
                                              const int* cu_seqlens, const int* seq_slot, const int* seq_start,
                                              const int* block_table, int max_blocks, int n_blocks, int n_tokens,
                                              int n_seqs, int max_new, int n_heads, int n_kv_heads, int head_dim,
-                                             float scale, int* error_flag, cudaStream_t stream) {
+                                             float scale, int* error_flag, const float* sinks, int window,
+                                             int mask_chunk, cudaStream_t stream) {
   if (n_seqs < 0 || max_new < 0 || n_tokens < 0 || n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0 ||
       n_blocks <= 0)
     return XRT_ERR_ARGUMENT;
@@ -405,6 +420,6 @@ XRT_EXPORT int xrt_attention_prefill_tcgen05(void* out, const void* q, const voi
   // run beside the kernel before it, and the early launch was measured slower (28.2 against 27.8 ms a prompt of 2,048)
   xrt::attention_prefill_tcgen05_kernel<1><<<grid, 64 + 128, xrt::fa_smem_bytes(1), stream>>>(
       map_q, map_k, map_v, (__nv_bfloat16*)out, cu_seqlens, seq_slot, seq_start, block_table, max_blocks, n_heads,
-      n_kv_heads, scale * 1.4426950408889634f, error_flag);
+      n_kv_heads, scale * 1.4426950408889634f, error_flag, xrt::key_range(window, mask_chunk), sinks);
   return xrt::launch_status();
 }

@@ -7,7 +7,7 @@
 //   kv head of query head h = h / (n_heads / n_kv_heads)                       :741
 //   s_j = dot(q, k_j) / sqrt(head_dim), j = 0 .. pos (the causal mask is the bound)  :506, 736-751
 //   online softmax: running maximum and sum, rescale on a new maximum, divide at the end  :514-574
-// `window` > 0 keeps only keys with pos - j < window (absent in the reference; 0 = all keys).
+// `range` (KeyRange in common.cuh, absent in the reference) keeps only the keys of a window or of a chunk of positions.
 // Further options on the scores, all 32-bit and all off at 0 (ScoreOptions in common.cuh): the first `keep_first`
 // keys of a sequence stay visible behind the window; s <- cap * tanh(s / cap); s <- s - slope_h * (pos - j) with
 // slope_h = 2^(-rate (h + 1) / n_heads).  `sink`: the softmax's denominator holds one more term exp(sink_score)
@@ -21,7 +21,7 @@ __global__ void attention_reference_kernel(
     TO* __restrict__ out, const TQ* __restrict__ q, const TC* __restrict__ k_pool,
     const TC* __restrict__ v_pool, const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
     const int* __restrict__ block_table, int max_blocks, int n_heads, int n_kv_heads, int head_dim,
-    float scale, int window, const ScoreOptions opt) {
+    float scale, const KeyRange range, const ScoreOptions opt) {
   extern __shared__ float q_staged[];  // [warps][head_dim]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
@@ -44,7 +44,7 @@ __global__ void attention_reference_kernel(
 #pragma unroll
   for (int j = 0; j < MAX_PER_LANE; ++j) acc[j] = 0.f;
   float running_max = -INFINITY, running_sum = 0.f;
-  const int first_key = window > 0 ? max(0, pos - window + 1) : 0;
+  const int first_key = range.first(pos);
   const int kept = min(opt.keep_first, first_key);  // keys [0, kept) lie behind the window and stay visible
   const float slope = opt.distance_rate > 0.f ? exp2f(-opt.distance_rate * (float)(head + 1) / (float)n_heads) : 0.f;
   const int* blocks = block_table + (size_t)slot * max_blocks;
@@ -85,7 +85,7 @@ __global__ void attention_reference_kernel(
   };
   for (int base = 0; base < kept; base += 32) tile_of_keys(base, 0, kept);
   for (int base = (first_key / 32) * 32; base <= pos; base += 32) tile_of_keys(base, first_key, pos + 1);
-  if (opt.sink) running_sum += expf(opt.sink_score - running_max);  // every token sees itself: the maximum is a number
+  if (opt.sink) running_sum += expf(sink_of(opt, head) - running_max);  // every token sees itself: the maximum is a number
   const float inv = 1.0f / running_sum;
 #pragma unroll
   for (int j = 0; j < MAX_PER_LANE; ++j) {
@@ -101,13 +101,15 @@ XRT_EXPORT int xrt_attention_reference(void* out, const void* q, const void* k_p
                                        const int* tok_slot, const int* tok_pos, const int* block_table,
                                        int max_blocks, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                                        float scale, int window, int keep_first, float softcap, float distance_rate,
-                                       int sink, float sink_score, int q_dtype, int cache_dtype, int out_dtype, cudaStream_t stream) {
+                                       int sink, float sink_score, const float* sinks, int mask_chunk, int q_dtype, int cache_dtype, int out_dtype, cudaStream_t stream) {
   xrt::ScoreOptions opt;
   opt.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
   opt.softcap = softcap;
   opt.distance_rate = distance_rate;
   opt.sink = sink;
   opt.sink_score = sink_score;
+  opt.sinks = sinks;
+  const xrt::KeyRange range = xrt::key_range(window, mask_chunk);
   if (n_tokens < 0 || n_heads <= 0 || n_kv_heads <= 0 || head_dim <= 0 || n_heads % n_kv_heads != 0)
     return XRT_ERR_ARGUMENT;
   if (head_dim > 1024) return XRT_ERR_UNSUPPORTED;
@@ -123,7 +125,7 @@ XRT_EXPORT int xrt_attention_reference(void* out, const void* q, const void* k_p
       XRT_DISPATCH_DTYPE(out_dtype, TO, {                                                                       \
         xrt::attention_reference_kernel<TQ, TC, TO, PER_LANE><<<grid, warps * 32, smem, stream>>>(              \
             (TO*)out, (const TQ*)q, (const TC*)k_pool, (const TC*)v_pool, tok_slot, tok_pos, block_table,       \
-            max_blocks, n_heads, n_kv_heads, head_dim, scale, window, opt);                                     \
+            max_blocks, n_heads, n_kv_heads, head_dim, scale, range, opt);                                     \
       });                                                                                                       \
     });                                                                                                         \
   })

@@ -53,14 +53,34 @@ struct RowScale {
   int parts = 0;
   int width = 1;
   float eps = 0.f;
-  int gate_act = 0;                 // of a gated product (mode 2): 0 silu, 1 the tanh form of gelu
+  // of a gated product (mode 2): 0 silu, 1 the tanh form of gelu, 2 a limited gate: with g = min(g, limit) and
+  // u = clamp(u, -limit, limit) the result is g * sigmoid(alpha g) * (u + 1)
+  int gate_act = 0;
+  float gate_limit = 0.f, gate_alpha = 0.f;
+  const float* gate_bias = nullptr; // or [gate rows | up rows]: added to both sums before the gate
+  int gate_up = 0;                  // where the up rows' biases begin
+};
+
+// What a caller of a gated product may add to its mode: biases and the constants of the limited gate (null: none).
+struct GateOptions {
+  const float* bias;  // float32 [2 * N]: the N gate rows', then the N up rows'
+  float limit, alpha;
 };
 
 // The launchers take the gate's activation in the bits of `mode` above the low four: mode 2 | (act << 4).
 inline bool split_gate_act(int& mode, RowScale& scale) {
   scale.gate_act = mode >> 4;
   mode &= 15;
-  return scale.gate_act == 0 || (scale.gate_act == 1 && mode == 2);
+  return scale.gate_act == 0 || (scale.gate_act <= 2 && mode == 2);
+}
+inline bool take_gate_options(const GateOptions* gate, int mode, int n, RowScale& scale) {
+  if (gate == nullptr) return scale.gate_act != 2;  // the limited gate has constants
+  if (mode != 2) return false;
+  scale.gate_bias = gate->bias;
+  scale.gate_up = n;
+  scale.gate_limit = gate->limit;
+  scale.gate_alpha = gate->alpha;
+  return true;
 }
 
 // What an attention layer may do to its scores beside the scale, the causal bound and the window (0 = off):
@@ -72,7 +92,34 @@ struct ScoreOptions {
   float distance_rate = 0.f;
   int sink = 0;            // the softmax's denominator holds one more term exp(sink_score) that has no value
   float sink_score = 0.f;
+  const float* sinks = nullptr;  // [n_heads], with sink: a head's own score instead of sink_score
 };
+
+__device__ __forceinline__ float sink_of(const ScoreOptions& opt, int head) {
+  return opt.sinks != nullptr ? opt.sinks[head] : opt.sink_score;
+}
+
+// Which keys at or before its own position a query sees (0 = no such bound): the `window` most recent ones, or those
+// of its own chunk of `chunk` positions, counted from position 0 of the sequence.  first(pos) never falls as pos grows,
+// so the range of a tile of queries begins where its first query's does.
+struct KeyRange {
+  int window = 0;
+  int chunk = 0;
+  __host__ __device__ __forceinline__ bool bounded() const { return window > 0 || chunk > 0; }
+  __device__ __forceinline__ int first(int pos) const {
+    int lo = 0;
+    if (window > 0) lo = max(0, pos + 1 - window);
+    if (chunk > 0) lo = max(lo, pos - pos % chunk);
+    return lo;
+  }
+};
+
+inline KeyRange key_range(int window, int chunk) {
+  KeyRange range;
+  range.window = window;
+  range.chunk = chunk;
+  return range;
+}
 
 __device__ __forceinline__ float to_float(float v) { return v; }
 __device__ __forceinline__ float to_float(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -86,6 +133,28 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
 // The gate of a gated feed-forward: silu, or (act 1) 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))).
 __device__ __forceinline__ float gelu_tanh_gate(float g) {
   return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+}
+
+// x * sigmoid(alpha x) for a result of type TO.  A bfloat16 result keeps 8 bits: the fast exponential and
+// division (2 ulp of 32-bit each) change none of them, and are a tenth of the instructions, which is
+// what an epilogue that runs once a block pays for (its code comes cold from the L2).
+template <typename TO> __device__ __forceinline__ float swish_for(float x, float alpha) { return x / (1.0f + expf(-alpha * x)); }
+template <> __device__ __forceinline__ float swish_for<__nv_bfloat16>(float x, float alpha) {
+  return __fdividef(x, 1.0f + __expf(-alpha * x));
+}
+
+// A gated feed-forward's hidden unit n from the two sums of its row pair, as RowScale says.
+template <typename TO>
+__device__ __forceinline__ float gated_unit(float g, float u, int n, const RowScale& s) {
+  if (s.gate_bias != nullptr) {
+    g += __ldg(s.gate_bias + n);
+    u += __ldg(s.gate_bias + s.gate_up + n);
+  }
+  if (s.gate_act == 2) {
+    g = fminf(g, s.gate_limit);
+    return swish_for<TO>(g, s.gate_alpha) * (fminf(fmaxf(u, -s.gate_limit), s.gate_limit) + 1.0f);
+  }
+  return (s.gate_act == 1 ? gelu_tanh_gate(g) : swish_for<TO>(g, 1.0f)) * u;
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

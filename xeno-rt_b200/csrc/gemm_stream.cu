@@ -225,8 +225,7 @@ gemm_stream_kernel(TO* __restrict__ out, const __nv_bfloat16* __restrict__ x, co
       const float first = total(rg) * inv;
       TO* dst = out + (size_t)m * ldo + row;
       if (MODE == 2)
-        *dst = from_float<TO>((scale.gate_act == 1 ? gelu_tanh_gate(first) : first / (1.0f + expf(-first))) *
-                              (total(ROW_GROUPS + rg) * inv));
+        *dst = from_float<TO>(gated_unit<float>(first, total(ROW_GROUPS + rg) * inv, row, scale));
       else if (MODE == 1) {
         const float updated = to_float(*dst) + first;
         *dst = from_float<TO>(updated);
@@ -347,13 +346,14 @@ XRT_EXPORT int xrt_gemm_stream_norm_blocks(int M, int N) {
 // Only for M <= 16 (one group of weight rows a block).
 // in_squares not null (modes 0 and 2): x is the result of such a product, residual * norm weight, and
 // in_squares = float32 [in_parts, M] the parts of its rows' sums of squares: every row of the result is
-// multiplied by 1 / sqrt(sum of the row's parts / K + eps).
+// multiplied by 1 / sqrt(sum of the row's parts / K + eps).  `gate` (may be null, a host structure): biases and the
+// constants of a limited gate with mode 2.
 XRT_EXPORT int xrt_gemm_stream_normed(void* out, const void* x, const void* w, int M, int N, int K, int ldx, int ldo,
                                       int out_dtype, int mode, int up_rows, void* scaled, int ld_scaled,
                                       const void* norm_weight, int norm_dtype, float* squares, const float* in_squares,
-                                      int in_parts, float eps, cudaStream_t stream) {
+                                      int in_parts, float eps, const xrt::GateOptions* gate, cudaStream_t stream) {
   xrt::RowScale scale;
-  if (mode < 0 || !xrt::split_gate_act(mode, scale)) return XRT_ERR_ARGUMENT;
+  if (mode < 0 || !xrt::split_gate_act(mode, scale) || !xrt::take_gate_options(gate, mode, N, scale)) return XRT_ERR_ARGUMENT;
   if (in_squares != nullptr && (in_parts <= 0 || mode == 1)) return XRT_ERR_ARGUMENT;
   scale.squares = in_squares; scale.parts = in_parts; scale.width = K; scale.eps = eps;
   if (M < 0 || N <= 0 || K <= 0 || ldx < K || ldo < N || mode < 0 || mode > 2) return XRT_ERR_ARGUMENT;
@@ -380,7 +380,7 @@ XRT_EXPORT int xrt_gemm_stream_norm(void* out, const void* x, const void* w, int
                                     int out_dtype, int mode, int up_rows, void* scaled, int ld_scaled,
                                     const void* norm_weight, int norm_dtype, float* squares, cudaStream_t stream) {
   return xrt_gemm_stream_normed(out, x, w, M, N, K, ldx, ldo, out_dtype, mode, up_rows, scaled, ld_scaled, norm_weight,
-                                norm_dtype, squares, nullptr, 0, 0.f, stream);
+                                norm_dtype, squares, nullptr, 0, 0.f, nullptr, stream);
 }
 
 // The same without a norm to prepare.

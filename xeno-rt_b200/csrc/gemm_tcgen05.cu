@@ -209,9 +209,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
           tmem_wait_ld();
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
-            const float g = __uint_as_float(v[j]) * row_inv;
-            const float a = scale.gate_act == 1 ? gelu_tanh_gate(g) : g / (1.0f + expf(-g));
-            v[j] = __float_as_uint(a * (__uint_as_float(u[j]) * row_inv));
+            // (columns beyond N are computed with the last one's bias and not stored)
+            v[j] = __float_as_uint(gated_unit<float>(__uint_as_float(v[j]) * row_inv, __uint_as_float(u[j]) * row_inv,
+                                                     min(col0 + c + j, N - 1), scale));
           }
         } else {
           tmem_wait_ld();
@@ -364,13 +364,15 @@ XRT_EXPORT int xrt_gemm_tcgen05_norm_parts(int N) { return N <= 0 ? XRT_ERR_ARGU
 // out) the product also writes (new out) * norm_weight there and the rows' sums of squares, one part a
 // tile of 256 columns, into squares = float32 [xrt_gemm_tcgen05_norm_parts(N), M].  With mode 0 or 2 and
 // in_squares not null (float32 [in_parts, M]) x is such a prepared input: row m of the result is
-// multiplied by 1 / sqrt(sum of the row's parts / K + eps).
+// multiplied by 1 / sqrt(sum of the row's parts / K + eps).  `gate` (may be null, a host structure): biases and the
+// constants of a limited gate with mode 2.
 XRT_EXPORT int xrt_gemm_tcgen05_normed(void* out, const void* x, const void* w, int M, int N, int K, int ldx, int ldo,
                                        int w_rows, int out_dtype, int mode, int up_rows, int* error_flag, void* scaled,
                                        int ld_scaled, const void* norm_weight, int norm_dtype, float* squares,
-                                       const float* in_squares, int in_parts, float eps, cudaStream_t stream) {
+                                       const float* in_squares, int in_parts, float eps, const xrt::GateOptions* gate,
+                                       cudaStream_t stream) {
   xrt::RowScale scale;
-  if (mode < 0 || !xrt::split_gate_act(mode, scale)) return XRT_ERR_ARGUMENT;
+  if (mode < 0 || !xrt::split_gate_act(mode, scale) || !xrt::take_gate_options(gate, mode, N, scale)) return XRT_ERR_ARGUMENT;
   if (M < 0 || N <= 0 || K <= 0 || ldx < K || ldo < N || mode < 0 || mode > 2) return XRT_ERR_ARGUMENT;
   if (mode == 1 && out_dtype != XRT_F32) return XRT_ERR_ARGUMENT;
   if (mode == 2 ? w_rows < up_rows + N : w_rows < N) return XRT_ERR_ARGUMENT;
@@ -416,5 +418,5 @@ XRT_EXPORT int xrt_gemm_tcgen05(void* out, const void* x, const void* w, int M, 
                                 int w_rows, int out_dtype, int mode, int up_rows, int* error_flag,
                                 cudaStream_t stream) {
   return xrt_gemm_tcgen05_normed(out, x, w, M, N, K, ldx, ldo, w_rows, out_dtype, mode, up_rows, error_flag, nullptr, 0,
-                                 nullptr, XRT_F32, nullptr, nullptr, 0, 0.f, stream);
+                                 nullptr, XRT_F32, nullptr, nullptr, 0, 0.f, nullptr, stream);
 }

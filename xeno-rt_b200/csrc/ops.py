@@ -29,7 +29,7 @@ _SIGNATURES = {
     "xrt_embedding": [_P, _P, _P, _I, _I, _I, _I, _P, _F, _P],
     "xrt_rmsnorm": [_P, _P, _P, _P, _I, _I, _F, _I, _I, _P],
     "xrt_layernorm": [_P, _P, _P, _P, _I, _I, _F, _I, _I, _P],
-    "xrt_swiglu": [_P, _P, _I, _I, _I, _I, _I, _P],
+    "xrt_swiglu": [_P, _P, _I, _I, _I, _I, _I, _P, _P],
     "xrt_rotation_table": [_P, _P, _P, _P, _F, _I, _I, _P],
     "xrt_state_scan": [_P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
     "xrt_removal_gates": [_P, _I, _P, _P, _I, _P, _P, _I, _P, _I, _I, _I, _I, _F, _F, _P],
@@ -67,24 +67,28 @@ _SIGNATURES = {
     "xrt_rope_table": [_P, _P, _P, _F, _I, _I, _P],
     "xrt_qk_rope_kv_write": [_P, _P, _P, _P, _I, _I, _I, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I,
                              _I, _I, _I, _I, _I, _P],
-    "xrt_attention_reference": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _I, _I, _I, _P],
+    "xrt_attention_reference": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _P, _I, _I, _I, _I, _P],
     "xrt_gemm_reference": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "xrt_gemm_stream": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "xrt_gemm_stream_norm": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _P, _P],
-    "xrt_gemm_stream_normed": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _P, _P, _I, _F, _P],
-    "xrt_gemm_tcgen05_normed": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _P, _P, _I, _F, _P],
-    "xrt_gemm_decode_tcgen05_normed": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P],
+    "xrt_gemm_stream_normed": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _I, _P, _P, _I, _F, _P, _P],
+    "xrt_gemm_tcgen05_normed": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _P, _P, _I, _F, _P, _P],
+    "xrt_gemm_decode_tcgen05_normed": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P, _P],
     "xrt_gemm_tcgen05": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "xrt_gemm_decode_tcgen05": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "xrt_gemm_decode_tcgen05_norm": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _P, _P],
     "xrt_gemm_decode_tcgen05_norm_parts": [_I, _I, _I, _I],
-    "xrt_attention_decode_fused": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _P, _I],
-    "xrt_attention_decode": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _P, _I],
+    "xrt_attention_decode_fused": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _P, _I, _P, _I],
+    "xrt_attention_decode": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _P, _I, _P, _I],
     "xrt_attention_decode_qkv": [_P, _P, _P, _P, _P, _I, _I, _I, _P, _P, _I, _F, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I,
-                                 _I, _I, _F, _I, _I, _I, _P, _P, _P, _I],
-    "xrt_attention_decode_scored": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _I, _I, _P],
-    "xrt_attention_prefill": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _P],
-    "xrt_attention_prefill_tcgen05": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P],
+                                 _I, _I, _F, _I, _I, _I, _P, _P, _P, _I, _P, _I],
+    "xrt_attention_decode_scored": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _P, _I, _I, _I, _P],
+    "xrt_attention_prefill": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _P, _I, _P],
+    "xrt_attention_prefill_tcgen05": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _I, _I, _P],
+    "xrt_recurrence_conv": [_P, _I, _P],
+    "xrt_recurrence_gates": [_P, _P, _P, _P, _P, _I, _P],
+    "xrt_recurrence_scan": [_P, _P, _I, _I, _P],
+    "xrt_recurrence_step": [_P, _P, _P, _P, _P, _P, _I, _P],
     "xrt_fill_normal": [_P, ctypes.c_longlong, ctypes.c_ulonglong, ctypes.c_double, ctypes.c_double, _I, _P],
     "xrt_sample": [_P, _P, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P],
     "xrt_mark_seen": [_P, _I, _P, _P, _I, _I, _P],
@@ -288,25 +292,54 @@ def layernorm(out, x, weight, eps: float, rows=None) -> None:
                                    _code(weight.dtype), _code(out.dtype), _stream()), "layernorm")
 
 
-GATE_ACTS = {"silu": 0, "gelu_tanh": 1}
+GATE_ACTS = {"silu": 0, "gelu_tanh": 1, "gated_sigmoid": 2}
 
 
-def _gate_code(act: str, mode: str) -> int:
-    """The number of a gated product's activation ("swiglu" mode only: silu, or the tanh form of gelu)."""
-    if act not in GATE_ACTS or (act != "silu" and mode != "swiglu"):
+class _GateOptions(ctypes.Structure):
+    _fields_ = [("bias", _P), ("limit", _F), ("alpha", _F)]
+
+
+@dataclasses.dataclass(frozen=True)
+class Gate:
+    """What a gated product does with its two sums g and u: ``act`` "silu" or "gelu_tanh" gives act(g) * u,
+    "gated_sigmoid" gives g * sigmoid(alpha g) * (u + 1) with g = min(g, limit) and u = clamp(u, -limit, limit).  ``bias``
+    (float32 [2 * width], the gate rows' and then the up rows', or None) is added to the sums first."""
+    act: str = "silu"
+    limit: float = 0.0
+    alpha: float = 0.0
+    bias: torch.Tensor | None = None
+
+    def options(self, width: int):
+        """The host structure that the launchers take, or None where there is nothing beyond ``act``."""
+        if self.bias is None and self.act != "gated_sigmoid":
+            return None
+        if self.bias is not None and self.bias.numel() != 2 * width:
+            raise KernelError("a gated product needs one bias a gate row and one an up row")
+        return ctypes.byref(_GateOptions(_ptr(self.bias, "bias", torch.float32), float(self.limit), float(self.alpha)))
+
+
+def _gate_of(act) -> Gate:
+    return act if isinstance(act, Gate) else Gate(act)
+
+
+def _gate_code(gate: Gate, mode: str) -> int:
+    """The number of a gated product's activation ("swiglu" mode only)."""
+    act = gate.act
+    if act not in GATE_ACTS or ((act != "silu" or gate.bias is not None) and mode != "swiglu"):
         raise KernelError(f"the gate's activation {act!r} is not one of {sorted(GATE_ACTS)}, or the product has no gate")
     return GATE_ACTS[act]
 
 
-def swiglu(out, gate_up, act: str = "silu") -> None:
-    """out[t, f] = act(gate_up[t, f]) * gate_up[t, F + f]; ``act`` "silu" or "gelu_tanh" (the tanh form of gelu)."""
-    if act not in GATE_ACTS:
-        raise KernelError(f"swiglu: the gate's activation {act!r} is not one of {sorted(GATE_ACTS)}")
+def swiglu(out, gate_up, act="silu") -> None:
+    """out[t, f] = act(gate_up[t, f]) * gate_up[t, F + f]; ``act`` "silu" or "gelu_tanh" (the tanh form of gelu), or a
+    ``Gate`` (a limited gate, biases)."""
+    gate = _gate_of(act)
+    code = _gate_code(gate, "swiglu")
     n, width = out.shape
     if gate_up.shape[0] != n or gate_up.shape[1] != 2 * width:
         raise KernelError("swiglu: shapes do not fit")
     _check(_kernels().xrt_swiglu(_ptr(out, "out"), _ptr(gate_up, "gate_up"), n, width, _code(gate_up.dtype),
-                                _code(out.dtype), GATE_ACTS[act], _stream()), "swiglu")
+                                _code(out.dtype), code, gate.options(width), _stream()), "swiglu")
 
 
 def rope_table(cos_sin, positions, freq, scale: float) -> None:
@@ -350,13 +383,29 @@ def qk_rope_kv_write(q_out, k_pool, v_pool, qkv, k_offset: int, v_offset: int, q
         _code(q_out.dtype), _code(cache_dtype), _stream()), "qk_rope_kv_write")
 
 
+def _sink_args(sink, n_heads: int) -> tuple:
+    """(on, one score for all heads, pointer to one score a head) of a softmax sink: None, a number or float32 [heads]."""
+    if sink is None:
+        return 0, 0.0, 0
+    if isinstance(sink, torch.Tensor):
+        return 1, 0.0, _sinks(sink, n_heads)
+    return 1, float(sink), 0
+
+
+def _sinks(sinks, n_heads: int) -> int:
+    if sinks is not None and sinks.numel() != n_heads:
+        raise KernelError("attention: one sink a head is needed")
+    return _ptr(sinks, "sinks", torch.float32)
+
+
 def attention_reference(out, q, k_pool, v_pool, tok_slot, tok_pos, block_table, n_heads: int, n_kv_heads: int,
                         head_dim: int, scale: float, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
-                        distance_rate: float = 0.0, sink: float | None = None) -> None:
+                        distance_rate: float = 0.0, sink=None, mask_chunk: int = 0) -> None:
     """Causal GQA attention over the cache, one warp per (token, head); any dtype.  ``keep_first``: so many first
     keys stay visible behind the window; ``softcap``: s <- cap tanh(s / cap); ``distance_rate`` r: head h's scores
-    lose 2^(-r (h + 1) / heads) for every position between query and key (each 0 = off); ``sink`` (None = off): the
-    softmax's denominator holds one more term exp(sink) that has no value."""
+    lose 2^(-r (h + 1) / heads) for every position between query and key (each 0 = off); ``sink`` (None = off, a number,
+    or float32 [heads], one a head): the softmax's denominator holds one more term exp(sink) that has no value;
+    ``mask_chunk`` (0 = off): a query sees only the keys of its own chunk of so many positions, counted from position 0."""
     n = q.shape[0]
     if q.shape != (n, n_heads * head_dim) or out.shape != q.shape:
         raise KernelError("attention_reference: shapes do not fit")
@@ -367,7 +416,7 @@ def attention_reference(out, q, k_pool, v_pool, tok_slot, tok_pos, block_table, 
         _ptr(tok_slot, "tok_slot", torch.int32), _ptr(tok_pos, "tok_pos", torch.int32),
         _ptr(block_table, "block_table", torch.int32), block_table.shape[1], n, n_heads, n_kv_heads, head_dim,
         float(scale), int(window), int(keep_first), float(softcap), float(distance_rate),
-        0 if sink is None else 1, float(sink or 0.0), _code(q.dtype), _code(k_pool.dtype), _code(out.dtype), _stream()),
+        *_sink_args(sink, n_heads), int(mask_chunk), _code(q.dtype), _code(k_pool.dtype), _code(out.dtype), _stream()),
         "attention_reference")
 
 
@@ -473,7 +522,7 @@ def gemm_decode_tcgen05_norm_parts(m: int, n: int, k: int, device) -> int:
 
 
 def gemm_decode_tcgen05(out, x, w, mode: str = "store", up_rows: int = 0, squares=None, eps: float = 0.0, norm=None,
-                        gate_act: str = "silu") -> None:
+                        gate_act="silu") -> None:
     """bfloat16 product for at most 128 rows on the tcgen05 tensor cores with swapped operands:
     the weight is streamed once by TMA, K is split across blocks and summed in split order.
     ``squares`` (float32 [parts, rows], from a product with ``norm=...``): ``x`` is a residual times
@@ -492,7 +541,9 @@ def gemm_decode_tcgen05(out, x, w, mode: str = "store", up_rows: int = 0, square
     if (n + 127) // 128 > _COUNTER_SLOTS:
         raise KernelError("gemm_decode_tcgen05: more tiles than counters")
     code = {"store": 0, "accumulate": 1, "swiglu": 2}[mode]
-    coded = code | (_gate_code(gate_act, mode) << 4)  # the gate's activation rides above the mode's four bits
+    gate = _gate_of(gate_act)
+    coded = code | (_gate_code(gate, mode) << 4)  # the gate's activation rides above the mode's four bits
+    options = gate.options(n)
     flag, counters, sms = device_state(x.device)
     lib = library()
     floats = lib.xrt_gemm_decode_tcgen05_scratch(m, n, k, code, sms)
@@ -514,7 +565,7 @@ def gemm_decode_tcgen05(out, x, w, mode: str = "store", up_rows: int = 0, square
     _check(lib.xrt_gemm_decode_tcgen05_normed(
         out.data_ptr(), x.data_ptr(), _ptr(w, "w"), _ptr(partial, "partial"), counters.data_ptr(), m, n, k, x.stride(0),
         out.stride(0), w.shape[0], _code(out.dtype), coded, up_rows, sms, flag.data_ptr(),
-        _ptr(squares, "squares", torch.float32), 0 if squares is None else squares.shape[0], float(eps), _stream()),
+        _ptr(squares, "squares", torch.float32), 0 if squares is None else squares.shape[0], float(eps), options, _stream()),
         "gemm_decode_tcgen05")
 
 
@@ -524,7 +575,7 @@ def gemm_tcgen05_norm_parts(n: int) -> int:
 
 
 def gemm_tcgen05(out, x, w, mode: str = "store", up_rows: int = 0, norm=None, squares=None, eps: float = 0.0,
-                 gate_act: str = "silu") -> None:
+                 gate_act="silu") -> None:
     """bfloat16 product for many rows on the tcgen05 tensor cores with TMA-fed operands; modes as
     for ``gemm_stream``.  ``norm`` = (scaled, weight, squares) with "accumulate": the product prepares the
     RMSNorm that follows it (as ``gemm_stream`` does; ``squares`` is float32 [gemm_tcgen05_norm_parts(n), m]).
@@ -539,7 +590,9 @@ def gemm_tcgen05(out, x, w, mode: str = "store", up_rows: int = 0, norm=None, sq
     if x.stride(1) != 1 or out.stride(1) != 1 or not x.is_cuda or not out.is_cuda:
         raise KernelError("gemm_tcgen05: rows must be contiguous and on a CUDA device")
     code = {"store": 0, "accumulate": 1, "swiglu": 2}[mode]
-    coded = code | (_gate_code(gate_act, mode) << 4)  # the gate's activation rides above the mode's four bits
+    gate = _gate_of(gate_act)
+    coded = code | (_gate_code(gate, mode) << 4)  # the gate's activation rides above the mode's four bits
+    options = gate.options(n)
     flag = error_flag(x.device)
     scaled = weight = emitted = None
     if norm is not None:
@@ -553,7 +606,7 @@ def gemm_tcgen05(out, x, w, mode: str = "store", up_rows: int = 0, norm=None, sq
         out.data_ptr(), x.data_ptr(), _ptr(w, "w"), m, n, k, x.stride(0), out.stride(0), w.shape[0], _code(out.dtype), coded,
         up_rows, flag.data_ptr(), _ptr(scaled, "scaled", torch.bfloat16), 0 if scaled is None else scaled.stride(0),
         _ptr(weight, "weight"), _code(weight.dtype) if weight is not None else 0, _ptr(emitted, "squares", torch.float32),
-        _ptr(squares, "squares", torch.float32), 0 if squares is None else squares.shape[0], float(eps), _stream()),
+        _ptr(squares, "squares", torch.float32), 0 if squares is None else squares.shape[0], float(eps), options, _stream()),
         "gemm_tcgen05")
 
 
@@ -569,7 +622,7 @@ def gemm_stream_norm_parts(m: int, n: int) -> int:
 
 
 def gemm_stream(out, x, w, mode: str = "store", up_rows: int = 0, norm=None, squares=None, eps: float = 0.0,
-                gate_act: str = "silu") -> None:
+                gate_act="silu") -> None:
     """bfloat16 product for at most 64 rows that streams the weight once; ``mode`` is "store",
     "accumulate" (into a float32 out) or "swiglu" (out[m, n] = silu(x . w[n]) * (x . w[n + up_rows])).
     ``norm`` = (scaled, weight, squares) with "accumulate" and at most 16 rows: the product also
@@ -587,13 +640,17 @@ def gemm_stream(out, x, w, mode: str = "store", up_rows: int = 0, norm=None, squ
     if x.stride(1) != 1 or out.stride(1) != 1 or not x.is_cuda or not out.is_cuda:
         raise KernelError("gemm_stream: rows must be contiguous and on a CUDA device")
     code = {"store": 0, "accumulate": 1, "swiglu": 2}[mode]
-    coded = code | (_gate_code(gate_act, mode) << 4)  # the gate's activation rides above the mode's four bits
-    if squares is not None:
-        if norm is not None or mode == "accumulate" or squares.dim() != 2 or squares.shape[1] != m or not squares.is_contiguous():
+    gate = _gate_of(gate_act)
+    coded = code | (_gate_code(gate, mode) << 4)  # the gate's activation rides above the mode's four bits
+    options = gate.options(n)
+    if squares is not None or options is not None:
+        if squares is not None and (norm is not None or mode == "accumulate" or squares.dim() != 2 or squares.shape[1] != m
+                                    or not squares.is_contiguous()):
             raise KernelError("gemm_stream: squares must be [parts, rows], and not with accumulate or a following norm")
         _check(_kernels().xrt_gemm_stream_normed(
             out.data_ptr(), x.data_ptr(), _ptr(w, "w"), m, n, k, x.stride(0), out.stride(0), _code(out.dtype), coded, up_rows,
-            0, 0, 0, 0, 0, _ptr(squares, "squares", torch.float32), squares.shape[0], float(eps), _stream()), "gemm_stream")
+            0, 0, 0, 0, 0, _ptr(squares, "squares", torch.float32), 0 if squares is None else squares.shape[0], float(eps),
+            options, _stream()), "gemm_stream")
         return
     if norm is None:
         _check(_kernels().xrt_gemm_stream(out.data_ptr(), x.data_ptr(), _ptr(w, "w"), m, n, k, x.stride(0), out.stride(0),
@@ -611,12 +668,13 @@ def gemm_stream(out, x, w, mode: str = "store", up_rows: int = 0, norm=None, squ
 
 def attention_decode(out, q, k_pool, v_pool, tok_slot, tok_pos, block_table, n_heads: int, n_kv_heads: int,
                      head_dim: int, scale: float, window: int, chunk: int, n_splits: int, fused: bool = True,
-                     clusters: bool = True) -> None:
+                     clusters: bool = True, sinks=None, mask_chunk: int = 0) -> None:
     """bfloat16 attention of one token a sequence over its cache blocks, split along the keys.
     ``fused``: the splits are merged by the last block of each (token, kv head) instead of by a
     second kernel (needs the device's tile counters; falls back when there are too many).
     ``clusters`` False: the splits never merge as thread-block clusters (for sequences of very unequal
-    lengths: a cluster holds its places until its longest block is done)."""
+    lengths: a cluster holds its places until its longest block is done).  ``sinks`` (float32 [heads] or None) and
+    ``mask_chunk`` as for ``attention_reference``."""
     n = q.shape[0]
     if q.shape != (n, n_heads * head_dim) or out.shape != q.shape or tok_slot.numel() != n or tok_pos.numel() != n:
         raise KernelError("attention_decode: shapes do not fit")
@@ -636,7 +694,7 @@ def attention_decode(out, q, k_pool, v_pool, tok_slot, tok_pos, block_table, n_h
             k_pool.shape[0], _ptr(tok_slot, "tok_slot", torch.int32), _ptr(tok_pos, "tok_pos", torch.int32),
             _ptr(block_table, "block_table", torch.int32), block_table.shape[1], n, n_heads, n_kv_heads, head_dim,
             float(scale), int(window), int(chunk), int(n_splits), flag.data_ptr(), _stream(), ctypes.byref(merged),
-            1 if clusters else 0), "attention_decode")
+            1 if clusters else 0, _sinks(sinks, n_heads), int(mask_chunk)), "attention_decode")
         if n_splits > 1 and not merged.value and n_splits > attention_decode_fused_max_splits(head_dim, n_heads // n_kv_heads):
             add_launches(1)  # too many splits for the merging block: the combine kernel ran
         return
@@ -646,7 +704,7 @@ def attention_decode(out, q, k_pool, v_pool, tok_slot, tok_pos, block_table, n_h
         k_pool.shape[0], _ptr(tok_slot, "tok_slot", torch.int32), _ptr(tok_pos, "tok_pos", torch.int32),
         _ptr(block_table, "block_table", torch.int32), block_table.shape[1], n, n_heads, n_kv_heads, head_dim,
         float(scale), int(window), int(chunk), int(n_splits), flag.data_ptr(), _stream(), ctypes.byref(merged),
-        1 if clusters else 0), "attention_decode")
+        1 if clusters else 0, _sinks(sinks, n_heads), int(mask_chunk)), "attention_decode")
     if n_splits > 1 and not merged.value:
         add_launches(1)  # the combine kernel
 
@@ -662,7 +720,7 @@ def attention_decode_takes_qkv(n_heads: int, n_kv_heads: int, head_dim: int, rop
 def attention_decode_qkv(out, qkv, k_offset: int, v_offset: int, q_norm_w, k_norm_w, eps: float, cos_sin, k_pool, v_pool,
                          tok_slot, tok_pos, block_table, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                          window: int, chunk: int, n_splits: int, write_kv: bool = True, fused: bool = True,
-                         clusters: bool = True) -> None:
+                         clusters: bool = True, sinks=None, mask_chunk: int = 0) -> None:
     """Decode attention straight from the 32-bit output of the q/k/v product: per-head norms, rotation,
     the newest key and value into the cache (unless ``write_kv`` is False) and attention over the cache
     in ONE kernel (csrc/attention_decode.cu).  ``qkv``: float32 [n, row] with q at 0, k at ``k_offset``,
@@ -691,7 +749,7 @@ def attention_decode_qkv(out, qkv, k_offset: int, v_offset: int, q_norm_w, k_nor
         _ptr(v_pool, "v_pool", torch.bfloat16), k_pool.shape[0], _ptr(tok_slot, "tok_slot", torch.int32),
         _ptr(tok_pos, "tok_pos", torch.int32), _ptr(block_table, "block_table", torch.int32), block_table.shape[1], n,
         n_heads, n_kv_heads, head_dim, float(scale), int(window), int(chunk), int(n_splits), flag.data_ptr(), _stream(),
-        ctypes.byref(merged), 1 if clusters else 0), "attention_decode_qkv")
+        ctypes.byref(merged), 1 if clusters else 0, _sinks(sinks, n_heads), int(mask_chunk)), "attention_decode_qkv")
     if n_splits > 1 and not merged.value and (
             not use_counters or n_splits > attention_decode_fused_max_splits(head_dim, n_heads // n_kv_heads)):
         add_launches(1)  # the combine kernel
@@ -708,9 +766,9 @@ def attention_decode_fused_max_splits(head_dim: int, group: int) -> int:
 
 def attention_prefill(out, q, k_pool, v_pool, cu_seqlens, seq_slot, seq_start, block_table, max_new: int,
                       n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int = 0, keep_first: int = 0,
-                      softcap: float = 0.0, distance_rate: float = 0.0, sink: float | None = None) -> None:
+                      softcap: float = 0.0, distance_rate: float = 0.0, sink=None, mask_chunk: int = 0) -> None:
     """bfloat16 causal attention of sequences laid end to end, each continuing at seq_start.  ``keep_first``,
-    ``softcap``, ``distance_rate``: the score options of ``attention_reference``."""
+    ``softcap``, ``distance_rate``, ``sink``, ``mask_chunk``: the score options of ``attention_reference``."""
     n = q.shape[0]
     n_seqs = seq_slot.numel()
     if q.shape != (n, n_heads * head_dim) or out.shape != q.shape or cu_seqlens.numel() != n_seqs + 1:
@@ -723,12 +781,12 @@ def attention_prefill(out, q, k_pool, v_pool, cu_seqlens, seq_slot, seq_start, b
         _ptr(seq_slot, "seq_slot", torch.int32), _ptr(seq_start, "seq_start", torch.int32),
         _ptr(block_table, "block_table", torch.int32), block_table.shape[1], n_seqs, int(max_new), n_heads,
         n_kv_heads, head_dim, float(scale), int(window), int(keep_first), float(softcap), float(distance_rate),
-        0 if sink is None else 1, float(sink or 0.0), _stream()), "attention_prefill")
+        *_sink_args(sink, n_heads), int(mask_chunk), _stream()), "attention_prefill")
 
 
 def attention_decode_scored(out, q, k_pool, v_pool, tok_slot, tok_pos, block_table, n_heads: int, n_kv_heads: int,
                             head_dim: int, scale: float, window: int, keep_first: int, softcap: float, distance_rate: float,
-                            chunk: int, n_splits: int, sink: float | None = None) -> None:
+                            chunk: int, n_splits: int, sink=None, mask_chunk: int = 0) -> None:
     """bfloat16 attention of single new tokens with the score options of ``attention_reference``; a token's visible
     keys (kept first keys, then the window) are cut into ``n_splits`` stretches of ``chunk`` keys (a multiple of 32)."""
     n = q.shape[0]
@@ -745,14 +803,16 @@ def attention_decode_scored(out, q, k_pool, v_pool, tok_slot, tok_pos, block_tab
         _ptr(k_pool, "k_pool", torch.bfloat16), _ptr(v_pool, "v_pool", torch.bfloat16),
         _ptr(tok_slot, "tok_slot", torch.int32), _ptr(tok_pos, "tok_pos", torch.int32),
         _ptr(block_table, "block_table", torch.int32), block_table.shape[1], n, n_heads, n_kv_heads, head_dim, float(scale),
-        int(window), int(keep_first), float(softcap), float(distance_rate), 0 if sink is None else 1, float(sink or 0.0),
+        int(window), int(keep_first), float(softcap), float(distance_rate), *_sink_args(sink, n_heads), int(mask_chunk),
         int(chunk), int(n_splits), _stream()),
         "attention_decode_scored")
 
 
 def attention_prefill_tcgen05(out, q, k_pool, v_pool, cu_seqlens, seq_slot, seq_start, block_table, max_new: int,
-                              n_heads: int, n_kv_heads: int, head_dim: int, scale: float) -> None:
-    """bfloat16 causal attention of sequences laid end to end on the tcgen05 tensor cores (head size 128)."""
+                              n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int = 0, sinks=None,
+                              mask_chunk: int = 0) -> None:
+    """bfloat16 causal attention of sequences laid end to end on the tcgen05 tensor cores (head size 128); ``sinks``
+    (float32 [heads] or None) and ``mask_chunk`` as for ``attention_reference``."""
     n = q.shape[0]
     n_seqs = seq_slot.numel()
     if q.shape != (n, n_heads * head_dim) or out.shape != q.shape or cu_seqlens.numel() != n_seqs + 1:
@@ -765,7 +825,8 @@ def attention_prefill_tcgen05(out, q, k_pool, v_pool, cu_seqlens, seq_slot, seq_
         _ptr(v_pool, "v_pool", torch.bfloat16), _ptr(cu_seqlens, "cu_seqlens", torch.int32),
         _ptr(seq_slot, "seq_slot", torch.int32), _ptr(seq_start, "seq_start", torch.int32),
         _ptr(block_table, "block_table", torch.int32), block_table.shape[1], k_pool.shape[0], n, n_seqs, int(max_new),
-        n_heads, n_kv_heads, head_dim, float(scale), flag.data_ptr(), _stream()), "attention_prefill_tcgen05")
+        n_heads, n_kv_heads, head_dim, float(scale), flag.data_ptr(), _sinks(sinks, n_heads), int(window), int(mask_chunk),
+        _stream()), "attention_prefill_tcgen05")
 
 
 def fill_normal(out, key: int, mean: float, std: float) -> None:
@@ -1377,3 +1438,116 @@ def add_scaled_parts(residual, parts, scales) -> None:
     _check(_kernels().xrt_add_scaled_parts(_ptr(residual, "residual", torch.float32), _ptr(parts, "parts", torch.float32),
                                           _ptr(scales, "scales", torch.float32), residual.numel(), parts.shape[0],
                                           _stream()), "add_scaled_parts")
+
+
+# ---------------------------------------------------------------------------------------------------
+# The gated linear recurrence a channel (csrc/linear_recurrence.cu)
+class _RecurrenceArgs(ctypes.Structure):
+    _fields_ = [("p", _P), ("p_stride", _I), ("x_offset", _I), ("y_bias", _P), ("x_bias", _P), ("conv_w", _P),
+                ("conv_b", _P), ("r_bias", _P), ("i_bias", _P), ("rate", _P), ("state", _P), ("ring", _P),
+                ("cu_seqlens", _P), ("seq_slot", _P), ("seq_start", _P), ("n_seqs", _I), ("width", _I), ("taps", _I),
+                ("blocks", _I), ("u", _P), ("ab", _P), ("tiles", _P), ("init", _P), ("n_tiles", _I)]
+
+
+RECURRENCE_TILE = 64  # tokens of a sequence that one block of the scan walks
+
+
+@dataclasses.dataclass(frozen=True)
+class RecurrenceWeights:
+    """What the recurrence's kernels read beside the step: biases of the branches [width], the convolution ([width,
+    taps], [width]), the gates' biases [width] and ``rate`` = -c softplus(lam) [width], all float32; ``blocks`` square
+    matrices a gate [blocks, size, size]."""
+    y_bias: torch.Tensor
+    x_bias: torch.Tensor
+    conv: torch.Tensor
+    conv_bias: torch.Tensor
+    r_bias: torch.Tensor
+    i_bias: torch.Tensor
+    rate: torch.Tensor
+    r: torch.Tensor
+    i: torch.Tensor
+
+    @property
+    def width(self) -> int:
+        return self.rate.numel()
+
+    @property
+    def taps(self) -> int:
+        return self.conv.shape[1]
+
+
+def _recurrence_args(p, w: RecurrenceWeights, state, ring, cu_seqlens, seq_slot, seq_start, **buffers):
+    width, taps, blocks = w.width, w.taps, w.r.shape[0]
+    pp, ps = _columns(p, "p", 2 * width)
+    for t in (w.y_bias, w.x_bias, w.conv_bias, w.r_bias, w.i_bias):
+        if t.numel() != width:
+            raise KernelError("recurrence: one bias a channel is needed")
+    if w.conv.shape != (width, taps) or w.r.shape != w.i.shape or w.r.shape[1] != w.r.shape[2] or blocks * w.r.shape[1] != width:
+        raise KernelError("recurrence: the convolution or the gates' matrices do not fit")
+    if state.dim() != 2 or state.shape[1] != width or (taps > 1 and tuple(ring.shape) != (state.shape[0], taps, width)):
+        raise KernelError("recurrence: the state must be [slots, width] and the ring [slots, taps, width]")
+    n_seqs = seq_slot.numel()
+    if cu_seqlens.numel() != n_seqs + 1 or seq_start.numel() != n_seqs:
+        raise KernelError("recurrence: cu_seqlens must hold one entry more than seq_slot and seq_start")
+    f32 = torch.float32
+    args = _RecurrenceArgs(
+        p=pp, p_stride=ps, x_offset=width, y_bias=_ptr(w.y_bias, "y_bias", f32), x_bias=_ptr(w.x_bias, "x_bias", f32),
+        conv_w=_ptr(w.conv, "conv", f32), conv_b=_ptr(w.conv_bias, "conv_bias", f32), r_bias=_ptr(w.r_bias, "r_bias", f32),
+        i_bias=_ptr(w.i_bias, "i_bias", f32), rate=_ptr(w.rate, "rate", f32), state=_ptr(state, "state", f32),
+        ring=_ptr(ring if taps > 1 else None, "ring", f32), cu_seqlens=_ptr(cu_seqlens, "cu_seqlens", torch.int32),
+        seq_slot=_ptr(seq_slot, "seq_slot", torch.int32), seq_start=_ptr(seq_start, "seq_start", torch.int32),
+        n_seqs=n_seqs, width=width, taps=taps, blocks=blocks)
+    for name, t in buffers.items():
+        if name == "n_tiles":
+            args.n_tiles = int(t)
+        else:
+            setattr(args, name, _ptr(t, name, f32))
+    return args
+
+
+def recurrence_tensor_cores(w: RecurrenceWeights) -> bool:
+    """Whether the kernels with the gates' products on the tensor cores (and the one-launch step) take these matrices."""
+    return w.r.dtype == torch.bfloat16 and w.r.shape[1] % 8 == 0 and w.r.data_ptr() % 16 == 0 and w.i.data_ptr() % 16 == 0
+
+
+def linear_recurrence(out, p, w: RecurrenceWeights, state, ring, cu_seqlens, seq_slot, seq_start, max_new: int) -> None:
+    """out[t] = S_t * gelu_tanh(y_t + y_bias) for p float32 rows [y | x] of 2 * width columns, where a channel's state
+    follows S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with u = conv(x + x_bias), a_t = exp(rate sigmoid(R u_t + r_bias)),
+    i_t = sigmoid(I u_t + i_bias), R and I a square matrix a block of channels; all 32-bit.  ``state`` float32 [slots,
+    width] and ``ring`` float32 [slots, taps, width] (the convolution's last inputs, position p at entry p % taps) are
+    read and left as the sequences' last; rows of no sequence are not written."""
+    n, width = out.shape
+    if p.shape[0] != n or width != w.width:
+        raise KernelError("linear_recurrence: shapes do not fit")
+    n_seqs, n_tiles = seq_slot.numel(), -(-int(max_new) // RECURRENCE_TILE)
+    empty = lambda *shape: torch.empty(shape, dtype=torch.float32, device=p.device)
+    u, ab = empty(n, width), empty(n, width, 2)
+    tiles, init = empty(n_seqs, n_tiles, width, 2), empty(n_seqs, width)  # held until the last launch
+    args = ctypes.byref(_recurrence_args(p, w, state, ring, cu_seqlens, seq_slot, seq_start, u=u, ab=ab, tiles=tiles,
+                                         init=init, n_tiles=n_tiles))
+    lib = _kernels()
+    _check(lib.xrt_recurrence_conv(args, int(max_new), _stream()), "recurrence_conv")
+    if recurrence_tensor_cores(w):
+        _check(lib.xrt_recurrence_gates(args, _ptr(w.r, "r"), _ptr(w.i, "i"), 0, 0, int(max_new), _stream()), "recurrence_gates")
+    else:
+        if w.r.dtype != torch.float32 or w.i.dtype != torch.float32:
+            raise KernelError("linear_recurrence: matrices that the tensor cores do not take must be float32")
+        size = w.r.shape[1]
+        r_raw, i_raw = empty(n, width), empty(n, width)
+        for raw, m in ((r_raw, w.r), (i_raw, w.i)):
+            head_product(raw, size, 0, u, size, 0, m, m.shape[0])
+        _check(lib.xrt_recurrence_gates(args, 0, 0, _ptr(r_raw, "r_raw"), _ptr(i_raw, "i_raw"), int(max_new), _stream()),
+               "recurrence_gates")
+    _check(lib.xrt_recurrence_scan(_ptr(out, "out"), args, int(max_new), _code(out.dtype), _stream()), "recurrence_scan")
+
+
+def linear_recurrence_step(out, p, w: RecurrenceWeights, state, ring, tok_slot, tok_pos, cu_seqlens, seq_slot, seq_start) -> None:
+    """``linear_recurrence`` for a step of one token a sequence, in one launch (out bfloat16; check
+    ``recurrence_tensor_cores`` first).  Rows of no sequence (slot -1) give zeros."""
+    n, width = out.shape
+    if p.shape[0] != n or width != w.width or tok_slot.numel() != n or tok_pos.numel() != n:
+        raise KernelError("linear_recurrence_step: shapes do not fit")
+    args = ctypes.byref(_recurrence_args(p, w, state, ring, cu_seqlens, seq_slot, seq_start))
+    _check(_kernels().xrt_recurrence_step(_ptr(out, "out", torch.bfloat16), args, _ptr(w.r, "r", torch.bfloat16),
+                                          _ptr(w.i, "i", torch.bfloat16), _ptr(tok_slot, "tok_slot", torch.int32),
+                                          _ptr(tok_pos, "tok_pos", torch.int32), n, _stream()), "recurrence_step")

@@ -5,5 +5,6 @@ from . import givopel  # registers Givopel
 from . import guzuvik  # registers Guzuvik
 from . import zogevik  # registers Zogevik
 from . import sofunex  # registers Sofunex
+from . import fadutar  # registers Fadutar
 
-__all__ = ["llama", "givopel", "guzuvik", "zogevik", "sofunex"]
+__all__ = ["llama", "givopel", "guzuvik", "zogevik", "sofunex", "fadutar"]

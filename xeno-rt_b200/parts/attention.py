@@ -38,6 +38,17 @@ def _pad_columns(w, heads: int, size: int, to: int):
     return out.reshape(w.shape[0], heads * to).contiguous()
 
 
+def sink_scores(params, weights, n_heads: int, device):
+    """The softmax's sink of a layer as float32 [heads], or None: ``sink`` in params is a number (the same for all
+    heads) or "learned" (the weight ``sink``)."""
+    sink = params.get("sink")
+    if sink is None:
+        return None
+    if sink == "learned":
+        return weights["sink"].to(torch.float32).reshape(n_heads).contiguous()
+    return torch.full((n_heads,), float(sink), dtype=torch.float32, device=device)
+
+
 class GroupedQueryAttention:
     """params: ``width`` (model width), ``n_heads``, ``n_kv_heads``, ``head_dim``, ``qk_norm``
     (bool), ``eps`` (of the head norms), ``window`` (None = all keys), ``position`` (a PartSpec-like
@@ -53,7 +64,8 @@ class GroupedQueryAttention:
     ``qk_norm`` = "whole" (q and k are RMS-normed over the whole projection, all heads of a token at once, weights
     ``q_norm`` [n_heads*head_dim] and ``k_norm`` [n_kv_heads*head_dim], before the rotation), ``sink`` (a number s: the
     softmax's denominator holds one more term exp(s) that has no value, so a head may give less than an average of
-    its values), ``own_kv`` = False (the layer has no k and v products, norms or cache of its own: it is scheduled
+    its values; "learned": a number a head, the weight ``sink`` [n_heads]), ``chunk`` (a query sees only the keys of its own
+    chunk of so many positions, counted from position 0 of the sequence), ``own_kv`` = False (the layer has no k and v products, norms or cache of its own: it is scheduled
     with ``cache_from`` and reads the keys and values another layer cached, with its own queries, window and scale),
     ``conv`` (a number of taps: q, k and v pass a short causal convolution over time a channel, weights ``q_conv``,
     ``k_conv``, ``v_conv`` [channels, taps], right after the product and its bias, before norms and rotation; the
@@ -119,6 +131,8 @@ class GroupedQueryAttention:
                            "v_conv": ((nkv * vd, taps), "vector")})
         if params.get("o_bias"):
             shapes["o_bias"] = ((d,), "vector")
+        if params.get("sink") == "learned":
+            shapes["sink"] = ((nh,), "vector")
         return shapes
 
     def __init__(self, params, weights, dtype: DType, device):
@@ -134,7 +148,8 @@ class GroupedQueryAttention:
         self.unit_norm = self._unit_norm(params)
         self.whole_norm = self._whole_norm(params)
         self.own_kv = bool(params.get("own_kv", True))
-        self.sink = None if params.get("sink") is None else float(params["sink"])
+        self.sinks = sink_scores(params, weights, self.n_heads, device)
+        self.chunk = int(params.get("chunk") or 0)
         if not self.own_kv and (params.get("bias") or params.get("value_blend")):
             raise Unsupported("a layer without keys and values of its own cannot have their biases or blend them")
         self.keep_first = int(params.get("keep_first") or 0) if self.window else 0
@@ -205,7 +220,7 @@ class GroupedQueryAttention:
         # ops.qkv_heads_write and attend with the kernels that take the score options
         self.plain_heads = (self.bias is None and not self.unit_norm and not self.whole_norm and not self.value_blend
                             and true_dim == self.head_dim and not self.taps and not self.v_unit)
-        self.plain_scores = not (self.keep_first or self.softcap or self.distance_rate) and self.sink is None
+        self.plain_scores = not (self.keep_first or self.softcap or self.distance_rate)
         position = params.get("position") or {"kind": "none", "params": {}}
         self.position = part_class("position", position["kind"])(position.get("params", {}), {}, dtype, device)
         rope_dim = getattr(self.position, "rope_dim", 0)
@@ -216,7 +231,9 @@ class GroupedQueryAttention:
         self.act_dtype = torch_dtype(dtype)
 
     def cache_need(self):
-        keys = KVNeed(self.n_kv_heads, self.head_dim, self.window, self.keep_first)
+        # a chunk's keys are among as many most recent ones: what lies behind those can be given back
+        bounds = [int(b) for b in (self.window, self.chunk) if b]
+        keys = KVNeed(self.n_kv_heads, self.head_dim, min(bounds) if bounds else None, self.keep_first)
         if self.taps > 1:  # the convolution's last taps - 1 inputs, one row of the q/k/v product each
             return [keys, StateNeed((self.taps - 1, self.q_width + 2 * self.kv_width), "float32")]
         return keys
@@ -277,7 +294,8 @@ class GroupedQueryAttention:
             from . import attention_bf16
             if attention_bf16.decode_from_qkv(attended, qkv, self.q_width, self.q_width + self.kv_width, self.q_norm,
                                               self.k_norm, self.eps, cos_sin, pairing, ctx, store, self.n_heads,
-                                              self.n_kv_heads, self.head_dim, self.scale, window, owns_cache):
+                                              self.n_kv_heads, self.head_dim, self.scale, window, owns_cache, self.sinks,
+                                              self.chunk):
                 qkv = None
         if qkv is not None:
             q = torch.empty((n, self.q_width), dtype=self.act_dtype, device=h.device)
@@ -311,15 +329,16 @@ class GroupedQueryAttention:
 
     def attend(self, out, q, ctx, store):
         window = int(self.window) if self.window else 0
-        options = {} if self.plain_scores else {"keep_first": self.keep_first, "softcap": self.softcap,
-                                                "distance_rate": self.distance_rate, "sink": self.sink}
+        options = {"mask_chunk": self.chunk}
+        if not self.plain_scores:
+            options.update(keep_first=self.keep_first, softcap=self.softcap, distance_rate=self.distance_rate)
         if self.dtype is DType.BF16:
             from . import attention_bf16
             if attention_bf16.run(out, q, ctx, store, self.n_heads, self.n_kv_heads, self.head_dim, self.scale,
-                                  window, **options):
+                                  window, sinks=self.sinks, **options):
                 return
         ops.attention_reference(out, q, store.k, store.v, ctx.tok_slot, ctx.tok_pos, store.block_table,
-                                self.n_heads, self.n_kv_heads, self.head_dim, self.scale, window, **options)
+                                self.n_heads, self.n_kv_heads, self.head_dim, self.scale, window, sink=self.sinks, **options)
 
 
 register_part("mixer", "attention", GroupedQueryAttention)

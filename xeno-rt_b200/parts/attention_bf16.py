@@ -74,7 +74,7 @@ def _decode_split_of(ctx, n_kv_heads: int, device, window: int = 0):
 
 
 def decode_from_qkv(out, qkv, k_offset, v_offset, q_norm, k_norm, eps, cos_sin, pairing, ctx, store, n_heads, n_kv_heads,
-                    head_dim, scale, window, write_kv) -> bool:
+                    head_dim, scale, window, write_kv, sinks=None, mask_chunk=0) -> bool:
     """A decode step's attention straight from the q/k/v product's output: the kernel does the head norms,
     the rotation and the cache write itself (one kernel and one boundary less a layer).  False where that
     kernel does not take the case; the caller then runs the rotation kernel and ``run``."""
@@ -82,11 +82,11 @@ def decode_from_qkv(out, qkv, k_offset, v_offset, q_norm, k_norm, eps, cos_sin, 
     if not (ctx.all_single and ctx.n_tokens <= 65535
             and ops.attention_decode_takes_qkv(n_heads, n_kv_heads, head_dim, rope_half, pairing)):
         return False
-    chunk, n_splits, clusters = _decode_split_of(ctx, n_kv_heads, qkv.device, window)
+    chunk, n_splits, clusters = _decode_split_of(ctx, n_kv_heads, qkv.device, window or mask_chunk)
     fused = ctx.n_tokens * n_kv_heads <= FUSED_COMBINE_MAX
     ops.attention_decode_qkv(out, qkv, k_offset, v_offset, q_norm, k_norm, eps, cos_sin, store.k, store.v, ctx.tok_slot,
                              ctx.tok_pos, store.block_table, n_heads, n_kv_heads, head_dim, scale, window, chunk, n_splits,
-                             write_kv=write_kv, fused=fused, clusters=clusters)
+                             write_kv=write_kv, fused=fused, clusters=clusters, sinks=sinks, mask_chunk=mask_chunk)
     return True
 
 
@@ -102,42 +102,48 @@ def scored_decode_split(n_tokens: int, n_kv_heads: int, context: int, window: in
 
 
 def run(out, q, ctx, store, n_heads, n_kv_heads, head_dim, scale, window, keep_first=0, softcap=0.0,
-        distance_rate=0.0, sink=None) -> bool:
+        distance_rate=0.0, sinks=None, mask_chunk=0) -> bool:
+    """``sinks``: float32 [heads] or None; ``mask_chunk``: a query sees its own chunk of so many positions (0: all).  A
+    chunk is a window as far as launch shapes go: a token sees at most so many keys, from some position inside a block."""
     if n_heads // n_kv_heads > 16 or head_dim > 256:
         return False
+    bound = min(b for b in (window, mask_chunk) if b) if window or mask_chunk else 0
     # the layer's score options: kernels that take them only
-    scored = bool(keep_first or softcap or distance_rate) or sink is not None
+    scored = bool(keep_first or softcap or distance_rate)
     if scored and ctx.all_single and head_dim % 8 == 0 and n_kv_heads <= 65535:
-        chunk, n_splits = scored_decode_split(ctx.n_tokens, n_kv_heads, context_bucket(ctx.max_context), window,
+        chunk, n_splits = scored_decode_split(ctx.n_tokens, n_kv_heads, context_bucket(ctx.max_context), bound,
                                               keep_first, ops.device_state(q.device)[2])
         ops.attention_decode_scored(out, q, store.k, store.v, ctx.tok_slot, ctx.tok_pos, store.block_table, n_heads,
                                     n_kv_heads, head_dim, scale, window, keep_first, softcap, distance_rate, chunk, n_splits,
-                                    sink=sink)
+                                    sink=sinks, mask_chunk=mask_chunk)
         return True
     if scored:
         if head_dim % 16 or ctx.n_seqs > 65535 or n_heads > 65535:
             return False
         ops.attention_prefill(out, q, store.k, store.v, ctx.cu_seqlens, ctx.seq_slot, ctx.seq_start,
                               store.block_table, ctx.max_new, n_heads, n_kv_heads, head_dim, scale, window,
-                              keep_first, softcap, distance_rate, sink=sink)
+                              keep_first, softcap, distance_rate, sink=sinks, mask_chunk=mask_chunk)
         return True
     if ctx.all_single and ctx.n_tokens <= 65535:
-        chunk, n_splits, clusters = _decode_split_of(ctx, n_kv_heads, q.device, window)
+        chunk, n_splits, clusters = _decode_split_of(ctx, n_kv_heads, q.device, bound)
         # few sequences: the last block of a (token, kv head) merges its splits (one launch less);
         # many: a second kernel merges them with more threads (measured faster from 8 sequences on)
         # (a group's partial results of more than FUSED_COMBINE_WIDTH numbers a split are too much for one block)
         fused = (ctx.n_tokens * n_kv_heads <= FUSED_COMBINE_MAX
                  and (n_heads // n_kv_heads) * head_dim <= FUSED_COMBINE_WIDTH)
         ops.attention_decode(out, q, store.k, store.v, ctx.tok_slot, ctx.tok_pos, store.block_table, n_heads,
-                             n_kv_heads, head_dim, scale, window, chunk, n_splits, fused=fused, clusters=clusters)
+                             n_kv_heads, head_dim, scale, window, chunk, n_splits, fused=fused, clusters=clusters, sinks=sinks,
+                             mask_chunk=mask_chunk)
         return True
     if ctx.n_seqs <= 65535 and n_heads <= 65535:
-        if (head_dim == 128 and window == 0 and ctx.max_new >= TCGEN05_MIN_NEW
+        if (head_dim == 128 and scale > 0 and ctx.max_new >= TCGEN05_MIN_NEW
                 and ops.tuning().prefill_attention != "mma"):
             ops.attention_prefill_tcgen05(out, q, store.k, store.v, ctx.cu_seqlens, ctx.seq_slot, ctx.seq_start,
-                                          store.block_table, ctx.max_new, n_heads, n_kv_heads, head_dim, scale)
+                                          store.block_table, ctx.max_new, n_heads, n_kv_heads, head_dim, scale, window,
+                                          sinks, mask_chunk)
             return True
         ops.attention_prefill(out, q, store.k, store.v, ctx.cu_seqlens, ctx.seq_slot, ctx.seq_start,
-                              store.block_table, ctx.max_new, n_heads, n_kv_heads, head_dim, scale, window)
+                              store.block_table, ctx.max_new, n_heads, n_kv_heads, head_dim, scale, window,
+                              sink=sinks, mask_chunk=mask_chunk)
         return True
     return False

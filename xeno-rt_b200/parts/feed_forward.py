@@ -8,13 +8,17 @@ import torch
 from ..core import ConfigError, DType, torch_dtype
 from ..csrc import ops
 from .linear import linear
+from .norm import WeightedParts
 from .registry import register_part
 
 
 class SwiGLUFeedForward:
     """params: ``width``, ``inner`` (the feed-forward width); optional ``activation`` of the gate: "silu" (default) or
-    "gelu_tanh" (the tanh form of gelu: down( gelu_tanh(gate(h)) * up(h) )).
-    weights: ``gate``, ``up`` [inner, width], ``down`` [width, inner]."""
+    "gelu_tanh" (the tanh form of gelu: down( gelu_tanh(gate(h)) * up(h) )), or "gated_sigmoid" with ``limit`` and ``alpha``
+    (the hidden units of ``RoutedExperts``: g = min(gate(h), limit), u = clamp(up(h), -limit, limit),
+    g * sigmoid(alpha g) * (u + 1)); ``bias`` (bool: all three products have one).
+    weights: ``gate``, ``up`` [inner, width], ``down`` [width, inner], with biases ``gate_bias``, ``up_bias`` [inner],
+    ``down_bias`` [width]."""
 
     graph_safe = True
 
@@ -26,7 +30,10 @@ class SwiGLUFeedForward:
     @classmethod
     def weight_shapes(cls, params):
         d, f = params["width"], params["inner"]
-        return {"gate": ((f, d), "matrix"), "up": ((f, d), "matrix"), "down": ((d, f), "matrix")}
+        shapes = {"gate": ((f, d), "matrix"), "up": ((f, d), "matrix"), "down": ((d, f), "matrix")}
+        if params.get("bias"):
+            shapes.update({"gate_bias": ((f,), "vector"), "up_bias": ((f,), "vector"), "down_bias": ((d,), "vector")})
+        return shapes
 
     def __init__(self, params, weights, dtype: DType, device):
         self.width = int(params["width"])
@@ -40,10 +47,17 @@ class SwiGLUFeedForward:
         self.activation = params.get("activation", "silu")
         if self.activation not in ops.GATE_ACTS:
             raise ConfigError(f"the gate's activation {self.activation!r} is not one of {sorted(ops.GATE_ACTS)}")
+        bias = self.down_bias = None
+        if params.get("bias"):  # 32-bit, added to the products' 32-bit sums
+            bias = torch.cat([weights[r].to(torch.float32) for r in ("gate_bias", "up_bias")]).contiguous()
+            self.down_bias = weights["down_bias"].to(torch.float32).contiguous()
+        self.gate = ops.Gate(self.activation, float(params.get("limit") or 0.0), float(params.get("alpha") or 0.0), bias)
+        if self.activation == "gated_sigmoid" and not (self.gate.limit > 0 and self.gate.alpha > 0):
+            raise ConfigError("a limited gate needs a positive limit and alpha")
 
     def takes_pending_norm(self, rows: int, device) -> bool:
         """Whether the first product of ``forward`` can finish a norm that the part before prepared."""
-        if self.act_dtype != torch.bfloat16 or self.activation != "silu":
+        if self.act_dtype != torch.bfloat16 or self.activation != "silu" or self.gate.bias is not None:
             return False
         from . import linear_bf16
         return linear_bf16.takes_pending(rows, self.inner, self.width, "swiglu", device)
@@ -53,19 +67,28 @@ class SwiGLUFeedForward:
         fused = False
         if self.act_dtype == torch.bfloat16 and h.dtype == torch.bfloat16:
             from . import linear_bf16
-            fused = linear_bf16.run_swiglu(act, h, self.w_gate_up, self.inner, self.activation)
+            fused = linear_bf16.run_swiglu(act, h, self.w_gate_up, self.inner, self.gate)
         if not fused:
             gate_up = linear(h, self.w_gate_up, out_dtype=torch.float32)
-            ops.swiglu(act, gate_up, self.activation)
+            ops.swiglu(act, gate_up, self.gate)
         return act
 
     def apply(self, h, ctx, out=None):
-        """The result handed back, float32 [T, width] (written into ``out`` where that is given)."""
+        """The result handed back, float32 [T, width] (written into ``out`` where that is given; without ``out`` a part with
+        biases hands its last product back with the bias row still to be added, as ``WeightedParts``)."""
         ctx.then_norm = None
-        return linear(self._act(h), self.w_down, out_dtype=torch.float32, out=out)
+        y = linear(self._act(h), self.w_down, out_dtype=torch.float32, out=out)
+        if self.down_bias is None:
+            return y
+        if out is None:
+            return WeightedParts(y, bias=self.down_bias)
+        ops.add_row(y, self.down_bias)
+        return y
 
     def forward(self, h, residual, ctx):
         act = self._act(h)
+        if self.down_bias is not None:
+            ops.add_row(residual, self.down_bias)
         # the last product may prepare the norm that follows this part (ctx.then_norm, see parts/context.py)
         if getattr(ctx, "then_norm", None) is not None:
             _, ctx.pending = linear(act, self.w_down, accumulate_into=residual, then_norm=ctx.then_norm)

@@ -18,6 +18,7 @@ import torch
 from ..cache import KVNeed
 from ..core import ConfigError, DType, Unsupported, torch_dtype
 from ..csrc import ops
+from .attention import sink_scores
 from .linear import linear
 from .registry import part_class, register_part
 
@@ -25,7 +26,8 @@ from .registry import part_class, register_part
 class LatentAttention:
     """params: ``width``, ``n_heads``, ``head_dim`` (a head's plain query/key size), ``rot_dim`` (its rotated size),
     ``v_head_dim``, ``kv_rank`` (the latent's size), ``eps`` (of the latent's norm), ``scale``, ``window`` (None = all
-    keys), ``position`` (``{"kind", "params"}`` of a position part over ``rot_dim`` dims).
+    keys), ``position`` (``{"kind", "params"}`` of a position part over ``rot_dim`` dims), optional ``sink`` (a number, or
+    "learned" with a weight ``sink`` [n_heads]: one more term exp(sink) of the softmax's denominator that has no value).
     weights: ``q`` [n_heads*(head_dim+rot_dim), width], ``down`` [kv_rank+rot_dim, width], ``down_norm`` [kv_rank],
     ``up_k`` [n_heads*head_dim, kv_rank], ``up_v`` [n_heads*v_head_dim, kv_rank], ``o`` [width, n_heads*v_head_dim]."""
 
@@ -40,9 +42,12 @@ class LatentAttention:
     def weight_shapes(cls, params):
         d, nh = params["width"], params["n_heads"]
         hd, rd, vd, rank = params["head_dim"], params["rot_dim"], params["v_head_dim"], params["kv_rank"]
-        return {"q": ((nh * (hd + rd), d), "matrix"), "down": ((rank + rd, d), "matrix"),
-                "down_norm": ((rank,), "vector"), "up_k": ((nh * hd, rank), "matrix"),
-                "up_v": ((nh * vd, rank), "matrix"), "o": ((d, nh * vd), "matrix")}
+        shapes = {"q": ((nh * (hd + rd), d), "matrix"), "down": ((rank + rd, d), "matrix"),
+                  "down_norm": ((rank,), "vector"), "up_k": ((nh * hd, rank), "matrix"),
+                  "up_v": ((nh * vd, rank), "matrix"), "o": ((d, nh * vd), "matrix")}
+        if params.get("sink") == "learned":
+            shapes["sink"] = ((nh,), "vector")
+        return shapes
 
     def __init__(self, params, weights, dtype: DType, device):
         self.width = int(params["width"])
@@ -68,6 +73,7 @@ class LatentAttention:
         self.w_uk_t = weights["up_k"].reshape(self.n_heads, self.dim, self.rank).transpose(1, 2).contiguous()
         self.w_uv = weights["up_v"].reshape(self.n_heads, self.vdim, self.rank).contiguous()
         self.w_o = weights["o"]
+        self.sinks = sink_scores(params, weights, self.n_heads, device)
         position = params.get("position") or {"kind": "none", "params": {}}
         self.position = part_class("position", position["kind"])(position.get("params", {}), {}, dtype, device)
         if self.rot and getattr(self.position, "rope_dim", 0) != self.rot:
@@ -100,13 +106,15 @@ class LatentAttention:
             ops.head_product(q, self.head_size, 0, qd, self.dim + self.rot, first * (self.dim + self.rot),
                              self.w_uk_t[first:first + heads], heads)
             latent = (torch.zeros if padded else torch.empty)(q.shape, dtype=self.act_dtype, device=h.device)
+            sinks = None if self.sinks is None else self.sinks[first:first + heads]
             done = False
             if self.dtype is DType.BF16:
                 from . import attention_bf16
-                done = attention_bf16.run(latent, q, ctx, store, heads, 1, self.head_size, self.scale, window)
+                done = attention_bf16.run(latent, q, ctx, store, heads, 1, self.head_size, self.scale, window,
+                                          sinks=sinks)
             if not done:
                 ops.attention_reference(latent, q, store.k, store.v, ctx.tok_slot, ctx.tok_pos, store.block_table, heads,
-                                        1, self.head_size, self.scale, window)
+                                        1, self.head_size, self.scale, window, sink=sinks)
             ops.head_product(out, self.vdim, first * self.vdim, latent, self.head_size, 0, self.w_uv[first:first + heads],
                              heads)
         return out

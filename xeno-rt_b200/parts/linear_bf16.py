@@ -72,7 +72,7 @@ def _decode_kernel(rows: int, n: int, k: int, mode: str, device) -> str:
     return "tcgen05" if tcgen05_for_few_rows(sms, rows, n, k, mode) else "stream"
 
 
-def _product(out, x, weight, mode: str, up_rows: int = 0, gate_act: str = "silu") -> None:
+def _product(out, x, weight, mode: str, up_rows: int = 0, gate_act="silu") -> None:
     rows = x.shape[0]
     if rows > ops.DECODE_TCGEN05_MAX_ROWS:
         ops.gemm_tcgen05(out, x, weight, mode, up_rows, gate_act=gate_act)
@@ -149,12 +149,13 @@ def run(out, x, weight, accumulate: bool) -> bool:
     return True
 
 
-def run_swiglu(out, x, weight_gate_up, inner: int, gate_act: str = "silu") -> bool:
-    """out = act(x . gate^T) * (x . up^T) for the fused weight [2 * inner, width], act = silu or ``gate_act``
-    "gelu_tanh"; False if no fused kernel takes the shape."""
+def run_swiglu(out, x, weight_gate_up, inner: int, gate_act="silu") -> bool:
+    """out = act(x . gate^T) * (x . up^T) for the fused weight [2 * inner, width], act = silu, ``gate_act`` "gelu_tanh" or
+    an ``ops.Gate``; False if no fused kernel takes the shape."""
     from .norm import PendingNorm
     if isinstance(x, PendingNorm):
-        if gate_act != "silu":
+        gate = gate_act if isinstance(gate_act, ops.Gate) else ops.Gate(gate_act)
+        if gate.act != "silu" or gate.bias is not None:
             return False
         run_pending(out, x, weight_gate_up, inner)
         return True

@@ -41,15 +41,17 @@ class PendingNorm:
 @dataclass
 class WeightedParts:
     """A sublayer's result that is still in parts: ``parts`` float32 [n, T, width], their sum sum_p scales[p] *
-    parts[p] + bias being the result (``scales`` float32 [n] on the device, ``bias`` float32 [width] or None).  The
+    parts[p] + bias being the result (``scales`` float32 [n] on the device or None for ones, ``bias`` float32 [width] or
+    None; a result in one piece may be [T, width]).  The
     norm that follows the sublayer adds them up in its own pass over the row."""
     parts: torch.Tensor
-    scales: torch.Tensor
+    scales: torch.Tensor | None = None
     bias: torch.Tensor | None = None
 
 
 class RMSNorm:
-    """params: ``width``, ``eps``; optional ``gain`` (a number g: ``add_into`` adds g times the norm; ``forward`` does
+    """params: ``width``, ``eps``; optional ``offset`` (the stored weight is a difference from this number: the norm
+    multiplies by offset + weight, a 32-bit sum) and ``gain`` (a number g: ``add_into`` adds g times the norm; ``forward`` does
     not use it).  weights: ``weight`` [width]."""
 
     graph_safe = True
@@ -62,6 +64,8 @@ class RMSNorm:
         self.width = int(params["width"])
         self.eps = float(params["eps"])
         self.weight = weights["weight"]
+        if params.get("offset"):
+            self.weight = (self.weight.to(torch.float32) + float(params["offset"])).contiguous()
         self.gain = float(params.get("gain") or 1.0)
         self.out_dtype = torch_dtype(dtype)
 

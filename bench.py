@@ -376,10 +376,31 @@ def sofunex_config(width: int, heads: int, kv_heads: int, head_dim: int, inner: 
             "layers": [{"type": "parallel", "mixer": mixer, "mlp": dense if i % 2 == 0 else moe} for i in range(layers)]}
 
 
+def fadutar_config(width: int, heads: int, kv_heads: int, head_dim: int, inner: int, layers: int, vocab: int) -> dict:
+    """A Fadutar model at the sizes of a dense decoder of that width: layers go recurrence, attention, recurrence, latent
+    attention, and again, the second and every later attention layer reading the keys and values of the first; every
+    layer with a dense feed-forward of ``inner``.  The recurrence has ``width`` channels in ``heads`` blocks and 4 taps;
+    attention ``heads`` x ``head_dim`` with ``kv_heads`` kv heads in chunks of 1,000 positions; latent attention ``heads``
+    heads of ``head_dim`` plain and 64 rotated dimensions over a latent of 192 (a cached row of 256), every earlier key."""
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+            "mask": {"size": 1000}}
+    latent = {"heads": heads, "dim": head_dim, "rot_dim": 64, "vdim": head_dim, "kv_rank": 192,
+              "scale": (head_dim + 64) ** -0.5, "rot": {"dims": 64, "base": 500000.0}}
+    recurrence = {"width": width, "blocks": heads, "conv": 4}
+    mlp = {"kind": "dense", "ff": inner, "limit": 7.0}
+    out = []
+    for i in range(layers):
+        kind, mixer = [("rglru", recurrence), ("attention", attn), ("rglru", recurrence), ("latent_attention", latent)][i % 4]
+        if kind == "attention" and i > 1:
+            mixer = dict(mixer, kv_from=1)
+        out.append({"type": kind, "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Fadutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": out}
+
+
 DESIGN_CONFIGS = {"givopel": givopel_config, "guzuvik": guzuvik_config, "zogevik": zogevik_config,
-                  "sofunex": sofunex_config}
+                  "sofunex": sofunex_config, "fadutar": fadutar_config}
 # the library's model that is closest to a design, timed beside it at equal sizes (besides the dense decoder)
-DESIGN_NEIGHBOUR = {"zogevik": "guzuvik", "sofunex": "givopel"}
+DESIGN_NEIGHBOUR = {"zogevik": "guzuvik", "sofunex": "givopel", "fadutar": "zogevik"}
 
 DESIGN_SIZES = {
     # name: (width, heads, kv heads, head size, feed-forward width, vocabulary)

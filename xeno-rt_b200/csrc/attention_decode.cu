@@ -285,7 +285,11 @@ attention_decode_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
                 n_kv_heads, head_dim, sinks);
 }
 
-// One warp per (token, head): merges the splits' partials in split order.
+// Merges the splits' partials in split order: a warp has one (token, head) and 64 of its dims.  A lane works out the
+// weight of one split (its maximum against the largest of all), 32 splits at a time; every lane then adds up its two
+// dims with several splits' loads in flight.  A split that holds no visible key was never written: its weight is 0 and
+// it is not read.
+constexpr int COMBINE_DIMS = 64;
 __global__ void attention_combine_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ part_o,
                                          const float* __restrict__ part_ml, const int* __restrict__ tok_slot,
                                          const int* __restrict__ tok_pos, int n_tokens, int n_heads, int head_dim,
@@ -293,48 +297,45 @@ __global__ void attention_combine_kernel(__nv_bfloat16* __restrict__ out, const 
                                          const float* __restrict__ sinks) {
   pdl_trigger();
   pdl_wait();
-  const int warp_global = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
-  if (warp_global >= n_tokens * n_heads) return;
-  const int tok = warp_global / n_heads;
-  __nv_bfloat16* dst = out + (size_t)warp_global * head_dim;
+  const int lane = threadIdx.x & 31, pieces = (head_dim + COMBINE_DIMS - 1) / COMBINE_DIMS;
+  const int warp_global = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  const int row = warp_global / pieces;  // (token, head)
+  if (row >= n_tokens * n_heads) return;
+  const int tok = row / n_heads, d = (warp_global - row * pieces) * COMBINE_DIMS + 2 * lane;
+  const bool mine = d < head_dim;  // head sizes are multiples of 16: both dims or none
+  __nv_bfloat162* dst = reinterpret_cast<__nv_bfloat162*>(out + (size_t)row * head_dim + d);
   if (tok_slot[tok] < 0) {
-    for (int d = lane; d < head_dim; d += 32) dst[d] = __float2bfloat16_rn(0.f);
+    if (mine) *dst = __floats2bfloat162_rn(0.f, 0.f);
     return;
   }
   const int len = tok_pos[tok] + 1;
   const int first_key = range.first(len - 1);
-  const size_t base = (size_t)warp_global * n_splits;
+  const size_t base = (size_t)row * n_splits;
+  auto of_split = [&](int s) {  // (maximum, sum) of a split
+    return s < n_splits && split_live(s, chunk, first_key, len) ? *reinterpret_cast<const float2*>(part_ml + (base + s) * 2)
+                                                               : make_float2(-INFINITY, 0.f);
+  };
   float m = -INFINITY;
-  for (int s = 0; s < n_splits; ++s) {
-    const bool live = split_live(s, chunk, first_key, len);
-    if (live) m = fmaxf(m, part_ml[(base + s) * 2]);
-  }
+  for (int s0 = 0; s0 < n_splits; s0 += 32) m = fmaxf(m, of_split(s0 + lane).x);
+  m = warp_max(m);
   float l = 0.f;
-  float acc[8];
-#pragma unroll
-  for (int j = 0; j < 8; ++j) acc[j] = 0.f;
-  // splits in order; loads are predicated rather than skipped so that several splits' loads are
-  // in flight at once (a dead split's partials are never read: they may hold anything)
-#pragma unroll 4
-  for (int s = 0; s < n_splits; ++s) {
-    const bool live = split_live(s, chunk, first_key, len);
-    const float ms = live ? part_ml[(base + s) * 2] : -INFINITY;
-    const float ls = live ? part_ml[(base + s) * 2 + 1] : 0.f;
-    const float f = ms == -INFINITY ? 0.f : exp2f(ms - m);
-    l += f * ls;
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int d = lane + 32 * j;
-      const float o = (live && d < head_dim) ? part_o[(base + s) * head_dim + d] : 0.f;
-      acc[j] += f * o;
+  float2 acc = make_float2(0.f, 0.f);
+  for (int s0 = 0; s0 < n_splits; s0 += 32) {
+    const float2 ml = of_split(s0 + lane);
+    const float weight = ml.x == -INFINITY ? 0.f : exp2f(ml.x - m);
+    l += warp_sum(weight * ml.y);
+    const int here = min(32, n_splits - s0);
+#pragma unroll 8
+    for (int s = 0; s < here; ++s) {
+      const float f = __shfl_sync(0xffffffffu, weight, s);
+      float2 o = make_float2(0.f, 0.f);
+      if (mine && f != 0.f) o = *reinterpret_cast<const float2*>(part_o + (base + s0 + s) * head_dim + d);
+      acc.x = fmaf(f, o.x, acc.x);
+      acc.y = fmaf(f, o.y, acc.y);
     }
   }
-  l += sink_term(sinks, warp_global - tok * n_heads, m);
-#pragma unroll
-  for (int j = 0; j < 8; ++j) {
-    const int d = lane + 32 * j;
-    if (d < head_dim) dst[d] = __float2bfloat16_rn(acc[j] / l);
-  }
+  l += sink_term(sinks, row - tok * n_heads, m);
+  if (mine) *dst = __floats2bfloat162_rn(acc.x / l, acc.y / l);
 }
 
 // The form with the heads as columns, fed by TMA: a cache block's keys and values for one kv head
@@ -981,7 +982,7 @@ static int attention_decode_impl(void* out, float* part_o, float* part_ml, const
   if (status != XRT_OK) return status;
   if (merged_out != nullptr) *merged_out = merged ? 1 : 0;
   if (n_splits > 1 && counters == nullptr && !merged) {
-    const int warps = n_tokens * n_heads;
+    const int warps = n_tokens * n_heads * ((head_dim + COMBINE_DIMS - 1) / COMBINE_DIMS);
     const int threads = warps <= 1024 ? 64 : 256;  // few rows: two warps a block, so that they spread over the multiprocessors
     launch_kernel(attention_combine_kernel, dim3((warps * 32 + threads - 1) / threads), dim3(threads), 0, stream, o,
                   (const float*)part_o, (const float*)part_ml, tok_slot, tok_pos, n_tokens, n_heads, head_dim, range,

@@ -143,18 +143,55 @@ template <> __device__ __forceinline__ float swish_for<__nv_bfloat16>(float x, f
   return __fdividef(x, 1.0f + __expf(-alpha * x));
 }
 
-// A gated feed-forward's hidden unit n from the two sums of its row pair, as RowScale says.
-template <typename TO>
-__device__ __forceinline__ float gated_unit(float g, float u, int n, const RowScale& s) {
+// COUNT hidden units of a gated feed-forward from the two sums of their row pairs, as RowScale says, into g: units n,
+// n + 1, .. with ALONG, else COUNT times unit n (of several tokens).  The kind of gate is chosen once for all of them, so
+// that their exponentials and divisions run side by side.  Units at or beyond gate_up (with biases: the product's
+// width) are not stored by anybody: they get some other unit's biases.
+template <typename TO, int COUNT, bool ALONG>
+__device__ __forceinline__ void gated_units(float (&g)[COUNT], float (&u)[COUNT], int n, const RowScale& s) {
   if (s.gate_bias != nullptr) {
-    g += __ldg(s.gate_bias + n);
-    u += __ldg(s.gate_bias + s.gate_up + n);
+    const float* up = s.gate_bias + s.gate_up;
+    if (!ALONG) {
+      const float bg = __ldg(s.gate_bias + n), bu = __ldg(up + n);
+#pragma unroll
+      for (int j = 0; j < COUNT; ++j) { g[j] += bg; u[j] += bu; }
+    } else if (COUNT % 4 == 0 && ((n | s.gate_up) & 3) == 0 && ((uintptr_t)s.gate_bias & 15) == 0) {
+#pragma unroll
+      for (int j = 0; j + 3 < COUNT; j += 4) {
+        const int at = min(n + j, s.gate_up - 4);
+        const float4 bg = __ldg(reinterpret_cast<const float4*>(s.gate_bias + at));
+        const float4 bu = __ldg(reinterpret_cast<const float4*>(up + at));
+        g[j] += bg.x; g[j + 1] += bg.y; g[j + 2] += bg.z; g[j + 3] += bg.w;
+        u[j] += bu.x; u[j + 1] += bu.y; u[j + 2] += bu.z; u[j + 3] += bu.w;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < COUNT; ++j) {
+        const int at = min(n + j, s.gate_up - 1);
+        g[j] += __ldg(s.gate_bias + at);
+        u[j] += __ldg(up + at);
+      }
+    }
   }
   if (s.gate_act == 2) {
-    g = fminf(g, s.gate_limit);
-    return swish_for<TO>(g, s.gate_alpha) * (fminf(fmaxf(u, -s.gate_limit), s.gate_limit) + 1.0f);
+    const float limit = s.gate_limit, alpha = s.gate_alpha;
+#pragma unroll
+    for (int j = 0; j < COUNT; ++j)
+      g[j] = swish_for<TO>(fminf(g[j], limit), alpha) * (fminf(fmaxf(u[j], -limit), limit) + 1.0f);
+  } else if (s.gate_act == 1) {
+#pragma unroll
+    for (int j = 0; j < COUNT; ++j) g[j] = gelu_tanh_gate(g[j]) * u[j];
+  } else {
+#pragma unroll
+    for (int j = 0; j < COUNT; ++j) g[j] = swish_for<TO>(g[j], 1.0f) * u[j];
   }
-  return (s.gate_act == 1 ? gelu_tanh_gate(g) : swish_for<TO>(g, 1.0f)) * u;
+}
+
+template <typename TO>
+__device__ __forceinline__ float gated_unit(float g, float u, int n, const RowScale& s) {
+  float gs[1] = {g}, us[1] = {u};
+  gated_units<TO, 1, false>(gs, us, n, s);
+  return gs[0];
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

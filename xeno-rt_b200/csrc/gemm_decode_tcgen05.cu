@@ -294,14 +294,15 @@ gemm_decode_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
             }
             // sixteen values worked out side by side (rows beyond M too: their stores are left out), so
             // that one element's exponential and division do not wait for the one before it
-            float val[16];
+            float val[16], up[16];
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const float inv = scaled ? row_inv[c + j] : 1.f;
               val[j] = __uint_as_float(v[j]) * inv;
-              if (MODE == 2) val[j] = gated_unit<TO>(val[j], __uint_as_float(u[j]) * inv, n, scale);
+              if (MODE == 2) up[j] = __uint_as_float(u[j]) * inv;
               if (MODE == 1) val[j] += old[j];
             }
+            if (MODE == 2) gated_units<TO, 16, false>(val, up, n, scale);
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               if (c + j < shape.M) out[(size_t)(c + j) * shape.ldo + n] = from_float<TO>(val[j]);
@@ -388,14 +389,15 @@ gemm_decode_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
                 for (int j = 0; j < 16; ++j)
                   old[j] = m0 + j < shape.M ? __ldcg(reinterpret_cast<const float*>(out) + (size_t)(m0 + j) * shape.ldo + n) : 0.f;
               }
-              float val[16];
+              float val[16], up[16];
 #pragma unroll
               for (int j = 0; j < 16; ++j) {
                 const float inv = scaled ? row_inv[m0 + j] : 1.f;
                 val[j] = sums[0][j] * inv;
-                if (MODE == 2) val[j] = gated_unit<TO>(val[j], sums[GROUPS - 1][j] * inv, n, scale);
+                if (MODE == 2) up[j] = sums[GROUPS - 1][j] * inv;
                 if (MODE == 1) val[j] += old[j];
               }
+              if (MODE == 2) gated_units<TO, 16, false>(val, up, n, scale);
 #pragma unroll
               for (int j = 0; j < 16; ++j)
                 if (m0 + j < shape.M) out[(size_t)(m0 + j) * shape.ldo + n] = from_float<TO>(val[j]);
@@ -470,9 +472,8 @@ gemm_decode_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
             float val[4] = {sums[u][0].x * inv, sums[u][0].y * inv, sums[u][0].z * inv, sums[u][0].w * inv};
             if (MODE == 2) {
               const float4 up = sums[u][GROUPS - 1];
-              const float ups[4] = {up.x * inv, up.y * inv, up.z * inv, up.w * inv};
-#pragma unroll
-              for (int j = 0; j < 4; ++j) val[j] = gated_unit<TO>(val[j], ups[j], n_of[u] + j, scale);
+              float ups[4] = {up.x * inv, up.y * inv, up.z * inv, up.w * inv};
+              gated_units<TO, 4, true>(val, ups, n_of[u], scale);
             }
             if (MODE == 1) { val[0] += old[u].x; val[1] += old[u].y; val[2] += old[u].z; val[3] += old[u].w; }
             store_four(out + (size_t)m_of[u] * shape.ldo + n_of[u], val);

@@ -225,7 +225,7 @@ gemm_stream_kernel(TO* __restrict__ out, const __nv_bfloat16* __restrict__ x, co
       const float first = total(rg) * inv;
       TO* dst = out + (size_t)m * ldo + row;
       if (MODE == 2)
-        *dst = from_float<TO>(gated_unit<float>(first, total(ROW_GROUPS + rg) * inv, row, scale));
+        *dst = from_float<TO>(gated_unit<TO>(first, total(ROW_GROUPS + rg) * inv, row, scale));
       else if (MODE == 1) {
         const float updated = to_float(*dst) + first;
         *dst = from_float<TO>(updated);

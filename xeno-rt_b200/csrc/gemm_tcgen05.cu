@@ -207,12 +207,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
           uint32_t u[32];
           tmem_ld32(u, tmem_row + TC_BN / 2 + c);
           tmem_wait_ld();
+          float g[32], up[32];
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
-            // (columns beyond N are computed with the last one's bias and not stored)
-            v[j] = __float_as_uint(gated_unit<float>(__uint_as_float(v[j]) * row_inv, __uint_as_float(u[j]) * row_inv,
-                                                     min(col0 + c + j, N - 1), scale));
+            g[j] = __uint_as_float(v[j]) * row_inv;
+            up[j] = __uint_as_float(u[j]) * row_inv;
           }
+          gated_units<TO, 32, true>(g, up, col0 + c, scale);
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(g[j]);
         } else {
           tmem_wait_ld();
           if (MODE == 0 && scale.squares != nullptr) {

@@ -41,12 +41,19 @@ struct RecurrenceArgs {
   int n_tiles;
 };
 
-__device__ __forceinline__ float lr_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+// The division and the root by the special-function unit (2^-22 and 2^-23 of the result).
+__device__ __forceinline__ float lr_sigmoid(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
+__device__ __forceinline__ float lr_sqrt(float x) {
+  float y;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
-// (a, b) of a channel from its gates before their sigmoids (biases added) and its u.
+// (a, b) of a channel from its gates before their sigmoids (biases added) and its u.  With m = a - 1 (which keeps its
+// digits where a is close to 1) 1 - a^2 = -m (2 + m).
 __device__ __forceinline__ float2 lr_step_of(float r_raw, float i_raw, float u, float rate) {
-  const float log_a = rate * lr_sigmoid(r_raw);
-  return make_float2(expf(log_a), sqrtf(-expm1f(2.0f * log_a)) * lr_sigmoid(i_raw) * u);
+  const float m = expm1f(rate * lr_sigmoid(r_raw));
+  return make_float2(1.0f + m, lr_sqrt(-m * (2.0f + m)) * lr_sigmoid(i_raw) * u);
 }
 
 // The convolution's input of position `pos` (channel c): of this step's tokens where pos >= start, else of the ring.
@@ -257,7 +264,7 @@ lr_gates_mma_kernel(const RecurrenceArgs a, const __nv_bfloat16* __restrict__ w_
 // One thread a channel, one tile of tokens a block.  Every block takes the state at its tile's start from what the tiles
 // before it do to the step's first state, in order.  The last tile's block leaves the sequence's state and ring.
 template <typename TO>
-__global__ void __launch_bounds__(128) lr_scan_kernel(TO* __restrict__ out, const RecurrenceArgs a) {
+__global__ void __launch_bounds__(128, 4) lr_scan_kernel(TO* __restrict__ out, const RecurrenceArgs a) {
   pdl_trigger();
   pdl_wait();
   const int s = blockIdx.z, tile = gridDim.y - 1 - blockIdx.y, slot = a.seq_slot[s];  // later tiles have more before them
@@ -277,11 +284,23 @@ __global__ void __launch_bounds__(128) lr_scan_kernel(TO* __restrict__ out, cons
   const float2* ab = a.ab + first * a.width + c;
   const float* y = a.p + first * a.p_stride + c;
   TO* o = out + first * a.width + c;
-#pragma unroll 8
-  for (int l = 0; l < n; ++l) {
-    const float2 v = ab[(size_t)l * a.width];
-    state = fmaf(v.x, state, v.y);
-    o[(size_t)l * a.width] = from_float<TO>(state * gelu_tanh_gate(y[(size_t)l * a.p_stride] + yb));
+  // several tokens' loads in flight: a load may not pass a store that could alias it, so they are all asked for before
+  // the first result is written
+  constexpr int AHEAD = 16;
+  for (int at = 0; at < n; at += AHEAD) {
+    float2 v[AHEAD];
+    float g[AHEAD];
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j) {
+      const bool live = at + j < n;
+      v[j] = live ? ab[(size_t)(at + j) * a.width] : make_float2(1.f, 0.f);
+      g[j] = live ? y[(size_t)(at + j) * a.p_stride] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j) {
+      state = fmaf(v[j].x, state, v[j].y);
+      if (at + j < n) o[(size_t)(at + j) * a.width] = from_float<TO>(state * gelu_tanh_gate(g[j] + yb));
+    }
   }
   if (l0 + n < len) return;
   a.state[(size_t)slot * a.width + c] = state;
@@ -296,16 +315,22 @@ __global__ void __launch_bounds__(128) lr_scan_kernel(TO* __restrict__ out, cons
 // Steps of one token a sequence, bfloat16 matrices: a block has 32 channels of one block of channels (a warp 8) and
 // both matrices' rows for them, and walks the step's rows 16 at a time.  The block's weights are asked for before the
 // wait for the kernel before it.  Convolution inputs of the whole block of channels are worked out by every block that
-// needs them (at most LR_STEP_K at a time, in shared memory).  Rows of no sequence (slot < 0) give zeros.
-constexpr int LR_STEP_K = 256, LR_STEP_LD = LR_STEP_K + 4, LR_STEP_ROWS = 16;
+// needs them (at most LR_STEP_K at a time, in shared memory), a thread a channel, several rows' loads in flight; what
+// the end needs (states, gate inputs, biases) is asked for before the products.  Rows of no sequence (slot < 0) give
+// zeros.  TAPS 0: any number up to LR_MAX_TAPS.
+constexpr int LR_STEP_K = 256, LR_STEP_LD = LR_STEP_K + 4, LR_STEP_ROWS = 16, LR_STEP_GROUP = 4;
+template <int TAPS>
 __global__ void __launch_bounds__(128)
 lr_step_kernel(__nv_bfloat16* __restrict__ out, const RecurrenceArgs a, const __nv_bfloat16* __restrict__ w_r,
                const __nv_bfloat16* __restrict__ w_i, const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
                int n_tokens, int size) {
+  constexpr int MOST = TAPS > 0 ? TAPS : LR_MAX_TAPS;
   __shared__ __align__(16) float us[LR_STEP_ROWS][LR_STEP_LD];
   __shared__ int slots[LR_STEP_ROWS], places[LR_STEP_ROWS];
+  __shared__ int entries[LR_STEP_ROWS][LR_MAX_TAPS];  // ring row of the input under each tap but the last (-1: before the start)
   pdl_trigger();
   const int block = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int taps = TAPS > 0 ? TAPS : a.taps;
   const int o_row = blockIdx.x * 32 + warp * 8;  // this warp's first channel inside the block of channels
   constexpr int PIECES = LR_STEP_K / 32;
   uint4 wr[PIECES], wi[PIECES];
@@ -321,33 +346,95 @@ lr_step_kernel(__nv_bfloat16* __restrict__ out, const RecurrenceArgs a, const __
     }
   };
   load_weights(0);
-  pdl_wait();
+  // the step's arrays were written before the step began, weights long before
+  const int o = o_row + 2 * t, c_own = block * size + o;  // this lane's two channels (sizes are multiples of 8)
+  const bool own = o < size;
+  float2 rb = make_float2(0.f, 0.f), ib = rb, yb = rb, xb = rb, rate = rb;
+  if (own) {
+    rb = *reinterpret_cast<const float2*>(a.r_bias + c_own); ib = *reinterpret_cast<const float2*>(a.i_bias + c_own);
+    yb = *reinterpret_cast<const float2*>(a.y_bias + c_own); xb = *reinterpret_cast<const float2*>(a.x_bias + c_own);
+    rate = *reinterpret_cast<const float2*>(a.rate + c_own);
+  }
   const bool one_stretch = size <= LR_STEP_K;
+  bool waited = false;
   for (int row0 = 0; row0 < n_tokens; row0 += LR_STEP_ROWS) {
+    const int n_rows = min(LR_STEP_ROWS, n_tokens - row0);
     __syncthreads();
     if (threadIdx.x < LR_STEP_ROWS) {
-      const bool live = row0 + threadIdx.x < n_tokens;
-      slots[threadIdx.x] = live ? tok_slot[row0 + threadIdx.x] : -1;
-      places[threadIdx.x] = live ? tok_pos[row0 + threadIdx.x] : 0;
+      const int r = threadIdx.x;
+      const int slot = r < n_rows ? tok_slot[row0 + r] : -1, pos = r < n_rows ? tok_pos[row0 + r] : 0;
+      slots[r] = slot;
+      places[r] = pos;
+      for (int j = 0; j + 1 < taps; ++j) {
+        const int p = pos - (taps - 1) + j;
+        entries[r][j] = p >= 0 && slot >= 0 ? slot * taps + p % taps : -1;
+      }
     }
     __syncthreads();
-    auto conv = [&](int r, int c) {  // u of row r, channel c (of all channels)
-      const int slot = slots[r], pos = places[r];
-      float acc = a.conv_b[c];
-      for (int j = 0; j < a.taps; ++j)
-        acc = fmaf(a.conv_w[(size_t)c * a.taps + j], lr_input(a, slot, row0 + r, pos, pos - (a.taps - 1) + j, c), acc);
-      return acc;
+    if (!waited) { pdl_wait(); waited = true; }
+    // u of rows r0 .. r0 + LR_STEP_GROUP and channel c of all channels
+    auto conv = [&](int r0, int c, float (&u)[LR_STEP_GROUP]) {
+      float in[LR_STEP_GROUP][MOST];
+      const float bias = a.x_bias[c];
+#pragma unroll
+      for (int i = 0; i < LR_STEP_GROUP; ++i) {
+        const bool live = slots[r0 + i] >= 0;
+#pragma unroll
+        for (int j = 0; j < MOST; ++j) {
+          in[i][j] = 0.f;
+          if (j == taps - 1) {
+            if (live) in[i][j] = a.p[(size_t)(row0 + r0 + i) * a.p_stride + a.x_offset + c] + bias;
+          } else if (j < taps - 1 && live) {
+            const int e = entries[r0 + i][j];
+            if (e >= 0) in[i][j] = a.ring[(size_t)e * a.width + c];
+          }
+        }
+      }
+      const float cb = a.conv_b[c];
+#pragma unroll
+      for (int i = 0; i < LR_STEP_GROUP; ++i) u[i] = cb;
+#pragma unroll
+      for (int j = 0; j < MOST; ++j) {
+        if (j < taps) {
+          const float w = a.conv_w[(size_t)c * taps + j];
+#pragma unroll
+          for (int i = 0; i < LR_STEP_GROUP; ++i) u[i] = fmaf(w, in[i][j], u[i]);
+        }
+      }
     };
+    // this lane's states and branches, rows g and g + 8
+    float2 st[2], yv[2], xv[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = g + 8 * h;
+      st[h] = yv[h] = xv[h] = make_float2(0.f, 0.f);
+      if (own && slots[r] >= 0) {
+        const float* row = a.p + (size_t)(row0 + r) * a.p_stride;
+        st[h] = make_float2(a.state[(size_t)slots[r] * a.width + c_own], a.state[(size_t)slots[r] * a.width + c_own + 1]);
+        yv[h] = make_float2(row[c_own], row[c_own + 1]);
+        xv[h] = make_float2(row[a.x_offset + c_own], row[a.x_offset + c_own + 1]);
+      }
+    }
     float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+    float2 u_own[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
     for (int k0 = 0; k0 < size; k0 += LR_STEP_K) {
       const int stretch = min(LR_STEP_K, (size - k0 + 31) / 32 * 32);
       if (k0 > 0) __syncthreads();
-      for (int e = threadIdx.x; e < LR_STEP_ROWS * stretch; e += 128) {
-        const int r = e / stretch, k = e - r * stretch;
-        us[r][k] = (slots[r] >= 0 && k0 + k < size) ? conv(r, block * size + k0 + k) : 0.f;
+      for (int k = threadIdx.x; k < stretch; k += 128) {
+#pragma unroll
+        for (int r0 = 0; r0 < LR_STEP_ROWS; r0 += LR_STEP_GROUP) {
+          float u[LR_STEP_GROUP] = {0.f, 0.f, 0.f, 0.f};
+          if (r0 < n_rows && k0 + k < size) conv(r0, block * size + k0 + k, u);
+#pragma unroll
+          for (int i = 0; i < LR_STEP_GROUP; ++i) us[r0 + i][k] = u[i];
+        }
       }
       if (!one_stretch) load_weights(k0);
       __syncthreads();
+      if (own && o >= k0 && o < k0 + LR_STEP_K) {  // two neighbours of one stretch: the stretch is even
+#pragma unroll
+        for (int h = 0; h < 2; ++h) u_own[h] = make_float2(us[g + 8 * h][o - k0], us[g + 8 * h][o - k0 + 1]);
+      }
 #pragma unroll
       for (int j = 0; j < PIECES; ++j) {
         if (32 * j < stretch) {
@@ -371,24 +458,28 @@ lr_step_kernel(__nv_bfloat16* __restrict__ out, const RecurrenceArgs a, const __
         }
       }
     }
+    if (!own) continue;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = g + (e >> 1) * 8, o = o_row + 2 * t + (e & 1);
-      if (row0 + r >= n_tokens || o >= size) continue;
-      const int c = block * size + o, slot = slots[r];
-      __nv_bfloat16* dst = out + (size_t)(row0 + r) * a.width + c;
+    for (int h = 0; h < 2; ++h) {
+      const int r = g + 8 * h, slot = slots[r];
+      if (r >= n_rows) continue;
+      __nv_bfloat162* dst = reinterpret_cast<__nv_bfloat162*>(out + (size_t)(row0 + r) * a.width + c_own);
       if (slot < 0) {
-        *dst = __float2bfloat16_rn(0.f);
+        *dst = __floats2bfloat162_rn(0.f, 0.f);
         continue;
       }
-      const float2 v = lr_step_of(acc[0][e] + a.r_bias[c], acc[1][e] + a.i_bias[c], conv(r, c), a.rate[c]);
-      float* st = a.state + (size_t)slot * a.width + c;
-      const float state = fmaf(v.x, *st, v.y);
-      *st = state;
-      const float* row = a.p + (size_t)(row0 + r) * a.p_stride;
-      if (a.taps > 1)
-        a.ring[((size_t)slot * a.taps + places[r] % a.taps) * a.width + c] = row[a.x_offset + c] + a.x_bias[c];
-      *dst = __float2bfloat16_rn(state * gelu_tanh_gate(row[c] + a.y_bias[c]));
+      const float2 v0 = lr_step_of(acc[0][2 * h] + rb.x, acc[1][2 * h] + ib.x, u_own[h].x, rate.x);
+      const float2 v1 = lr_step_of(acc[0][2 * h + 1] + rb.y, acc[1][2 * h + 1] + ib.y, u_own[h].y, rate.y);
+      const float2 s = make_float2(fmaf(v0.x, st[h].x, v0.y), fmaf(v1.x, st[h].y, v1.y));
+      float* state = a.state + (size_t)slot * a.width + c_own;
+      state[0] = s.x;
+      state[1] = s.y;
+      if (taps > 1) {
+        float* ring = a.ring + ((size_t)slot * taps + places[r] % taps) * a.width + c_own;
+        ring[0] = xv[h].x + xb.x;
+        ring[1] = xv[h].y + xb.y;
+      }
+      *dst = __floats2bfloat162_rn(s.x * gelu_tanh_gate(yv[h].x + yb.x), s.y * gelu_tanh_gate(yv[h].y + yb.y));
     }
   }
 }
@@ -462,10 +553,20 @@ XRT_EXPORT int xrt_recurrence_step(void* out, const xrt::RecurrenceArgs* args, c
   if (n_tokens < 0 || a.width <= 0 || a.blocks <= 0 || a.width % a.blocks || a.taps < 1 || (a.taps > 1 && a.ring == nullptr))
     return XRT_ERR_ARGUMENT;
   const int size = a.width / a.blocks;
-  if (size % 8 || a.taps > xrt::LR_MAX_TAPS || a.blocks > 65535 || (((uintptr_t)w_r | (uintptr_t)w_i) & 15))
+  if (size % 8 || a.taps > xrt::LR_MAX_TAPS || a.blocks > 65535 || (((uintptr_t)w_r | (uintptr_t)w_i) & 15) ||
+      (((uintptr_t)out | (uintptr_t)a.r_bias | (uintptr_t)a.i_bias | (uintptr_t)a.y_bias | (uintptr_t)a.x_bias | (uintptr_t)a.rate) & 7))
     return XRT_ERR_UNSUPPORTED;
   if (n_tokens == 0) return XRT_OK;
-  xrt::launch_kernel(xrt::lr_step_kernel, dim3((size + 31) / 32, a.blocks), dim3(128), 0, stream, (__nv_bfloat16*)out, a,
-                     (const __nv_bfloat16*)w_r, (const __nv_bfloat16*)w_i, tok_slot, tok_pos, n_tokens, size);
+#define XRT_LR_STEP(TAPS)                                                                                          \
+  xrt::launch_kernel(xrt::lr_step_kernel<TAPS>, dim3((size + 31) / 32, a.blocks), dim3(128), 0, stream,              \
+                     (__nv_bfloat16*)out, a, (const __nv_bfloat16*)w_r, (const __nv_bfloat16*)w_i, tok_slot, tok_pos, \
+                     n_tokens, size)
+  switch (a.taps) {
+    case 2: XRT_LR_STEP(2); break;
+    case 3: XRT_LR_STEP(3); break;
+    case 4: XRT_LR_STEP(4); break;
+    default: XRT_LR_STEP(0);
+  }
+#undef XRT_LR_STEP
   return xrt::launch_status();
 }

@@ -380,10 +380,11 @@ def fadutar_config(width: int, heads: int, kv_heads: int, head_dim: int, inner: 
     """A Fadutar model at the sizes of a dense decoder of that width: layers go recurrence, attention, recurrence, latent
     attention, and again, the second and every later attention layer reading the keys and values of the first; every
     layer with a dense feed-forward of ``inner``.  The recurrence has ``width`` channels in ``heads`` blocks and 4 taps;
-    attention ``heads`` x ``head_dim`` with ``kv_heads`` kv heads in chunks of 1,000 positions; latent attention ``heads``
-    heads of ``head_dim`` plain and 64 rotated dimensions over a latent of 192 (a cached row of 256), every earlier key."""
+    attention ``heads`` x ``head_dim`` with ``kv_heads`` kv heads in chunks of 1,500 positions (a token at context 4,096
+    sees 1,096 keys); latent attention ``heads`` heads of ``head_dim`` plain and 64 rotated dimensions over a latent of
+    192 (a cached row of 256), every earlier key."""
     attn = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
-            "mask": {"size": 1000}}
+            "mask": {"size": 1500}}
     latent = {"heads": heads, "dim": head_dim, "rot_dim": 64, "vdim": head_dim, "kv_rank": 192,
               "scale": (head_dim + 64) ** -0.5, "rot": {"dims": 64, "base": 500000.0}}
     recurrence = {"width": width, "blocks": heads, "conv": 4}

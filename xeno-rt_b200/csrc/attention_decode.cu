@@ -1006,15 +1006,18 @@ static int attention_decode_impl(void* out, float* part_o, float* part_ml, const
 // touched and no second kernel runs), else 0.  clusters = 0 keeps the splits from merging as clusters:
 // a cluster lives until its longest block is done, so where the sequences' lengths are far apart the
 // blocks of a short sequence's splits would hold their places for nothing.
+// sinks: float32 [n_heads] (one more term exp(sink) of a head's denominator that has no value) or null; mask_chunk > 0: a
+// query sees only the keys of its own chunk of so many positions (KeyRange; the splits then cover chunk + 63 keys).
 // This entry point merges the splits with a second kernel.
 XRT_EXPORT int xrt_attention_decode(void* out, float* part_o, float* part_ml, const void* q, const void* k_pool,
                                     const void* v_pool, int n_blocks, const int* tok_slot, const int* tok_pos,
                                     const int* block_table, int max_blocks, int n_tokens, int n_heads, int n_kv_heads,
                                     int head_dim, float scale, int window, int chunk, int n_splits, int* error_flag,
-                                    cudaStream_t stream, int* merged, int clusters, const float* sinks,
-                                    int mask_chunk) {
+                                    cudaStream_t stream, int* merged, int clusters,
+                                    const float* sinks, int mask_chunk) {
   return xrt::attention_decode_impl(out, part_o, part_ml, q, k_pool, v_pool, n_blocks, tok_slot, tok_pos, block_table,
-                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, xrt::key_range(window, mask_chunk), chunk, n_splits,
+                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale,
+                                    xrt::key_range(window, mask_chunk), chunk, n_splits,
                                     nullptr, error_flag, stream, merged, xrt::DecodeFusedInput(), clusters != 0, sinks);
 }
 
@@ -1025,11 +1028,12 @@ XRT_EXPORT int xrt_attention_decode_fused(void* out, float* part_o, float* part_
                                           const void* k_pool, const void* v_pool, int n_blocks, const int* tok_slot,
                                           const int* tok_pos, const int* block_table, int max_blocks, int n_tokens,
                                           int n_heads, int n_kv_heads, int head_dim, float scale, int window, int chunk,
-                                          int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters, const float* sinks,
-                                    int mask_chunk) {
+                                          int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters,
+                                    const float* sinks, int mask_chunk) {
   if (counters == nullptr) return XRT_ERR_ARGUMENT;
   return xrt::attention_decode_impl(out, part_o, part_ml, q, k_pool, v_pool, n_blocks, tok_slot, tok_pos, block_table,
-                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, xrt::key_range(window, mask_chunk), chunk, n_splits,
+                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale,
+                                    xrt::key_range(window, mask_chunk), chunk, n_splits,
                                     counters, error_flag, stream, merged, xrt::DecodeFusedInput(), clusters != 0, sinks);
 }
 
@@ -1046,8 +1050,8 @@ XRT_EXPORT int xrt_attention_decode_qkv(void* out, float* part_o, float* part_ml
                                         int write_kv, void* k_pool, void* v_pool, int n_blocks, const int* tok_slot,
                                         const int* tok_pos, const int* block_table, int max_blocks, int n_tokens,
                                         int n_heads, int n_kv_heads, int head_dim, float scale, int window, int chunk,
-                                        int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters, const float* sinks,
-                                    int mask_chunk) {
+                                        int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters,
+                                    const float* sinks, int mask_chunk) {
   if (qkv == nullptr || (q_norm_w == nullptr) != (k_norm_w == nullptr) || n_blocks <= 0) return XRT_ERR_ARGUMENT;
   if (norm_dtype != XRT_F32 && norm_dtype != XRT_BF16) return XRT_ERR_UNSUPPORTED;
   xrt::DecodeFusedInput fused;
@@ -1058,7 +1062,8 @@ XRT_EXPORT int xrt_attention_decode_qkv(void* out, float* part_o, float* part_ml
   fused.k_pool = write_kv ? (__nv_bfloat16*)k_pool : nullptr;
   fused.v_pool = write_kv ? (__nv_bfloat16*)v_pool : nullptr;
   return xrt::attention_decode_impl(out, part_o, part_ml, nullptr, k_pool, v_pool, n_blocks, tok_slot, tok_pos, block_table,
-                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale, xrt::key_range(window, mask_chunk), chunk, n_splits,
+                                    max_blocks, n_tokens, n_heads, n_kv_heads, head_dim, scale,
+                                    xrt::key_range(window, mask_chunk), chunk, n_splits,
                                     counters, error_flag, stream, merged, fused, clusters != 0, sinks);
 }
 

@@ -65,8 +65,9 @@ class GroupedQueryAttention:
     ``q_norm`` [n_heads*head_dim] and ``k_norm`` [n_kv_heads*head_dim], before the rotation), ``sink`` (a number s: the
     softmax's denominator holds one more term exp(s) that has no value, so a head may give less than an average of
     its values; "learned": a number a head, the weight ``sink`` [n_heads]), ``chunk`` (a query sees only the keys of its own
-    chunk of so many positions, counted from position 0 of the sequence), ``own_kv`` = False (the layer has no k and v products, norms or cache of its own: it is scheduled
-    with ``cache_from`` and reads the keys and values another layer cached, with its own queries, window and scale),
+    chunk of so many positions, counted from position 0 of the sequence), ``own_kv`` = False (the layer has no k and v
+    products, norms or cache of its own: it is scheduled with ``cache_from`` and reads the keys and values another layer
+    cached, with its own queries, window or chunk, sinks and scale),
     ``conv`` (a number of taps: q, k and v pass a short causal convolution over time a channel, weights ``q_conv``,
     ``k_conv``, ``v_conv`` [channels, taps], right after the product and its bias, before norms and rotation; the
     last taps - 1 rows of the product are state of the sequence, so the part then asks for a ``StateNeed`` beside

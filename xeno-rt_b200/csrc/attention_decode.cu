@@ -392,6 +392,7 @@ struct DecodeFusedInput {
   int norm_dtype = XRT_F32;
   float eps = 0.f;
   const float2* cos_sin = nullptr;   // [tokens, head_dim / 2] (cos, sin), or null: no rotation
+  QueryTemp temp;                    // of the queries, after norm and rotation
   __nv_bfloat16* k_pool = nullptr;   // null: the newest key and value are in the cache already (a layer that reads another's)
   __nv_bfloat16* v_pool = nullptr;
 };
@@ -547,10 +548,12 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           }
         }
     }
+    const float q_factor = fused.temp.at(len - 1);
 #pragma unroll
     for (int ks = 0; ks < D_TILES / 2; ++ks)
 #pragma unroll
-      for (int e = 0; e < 2; ++e) qb[ks][e] = g < group ? pack_bf16(x[ks][e][0], x[ks][e][1]) : 0u;
+      for (int e = 0; e < 2; ++e)
+        qb[ks][e] = g < group ? pack_bf16(x[ks][e][0] * q_factor, x[ks][e][1] * q_factor) : 0u;
     if (writes_newest) {
       // Warp 0: the newest key (head norm, rotation); warp 1: the newest value.  A lane holds dims
       // lane + 32 j; the rotation's partner of a dim is in the same lane.  Both go to the cache for the
@@ -1051,7 +1054,7 @@ XRT_EXPORT int xrt_attention_decode_qkv(void* out, float* part_o, float* part_ml
                                         const int* tok_pos, const int* block_table, int max_blocks, int n_tokens,
                                         int n_heads, int n_kv_heads, int head_dim, float scale, int window, int chunk,
                                         int n_splits, int* error_flag, cudaStream_t stream, int* merged, int clusters,
-                                    const float* sinks, int mask_chunk) {
+                                        const float* sinks, int mask_chunk, float temp_coef, int temp_every) {
   if (qkv == nullptr || (q_norm_w == nullptr) != (k_norm_w == nullptr) || n_blocks <= 0) return XRT_ERR_ARGUMENT;
   if (norm_dtype != XRT_F32 && norm_dtype != XRT_BF16) return XRT_ERR_UNSUPPORTED;
   xrt::DecodeFusedInput fused;
@@ -1059,6 +1062,7 @@ XRT_EXPORT int xrt_attention_decode_qkv(void* out, float* part_o, float* part_ml
   fused.row_stride = row_stride; fused.k_offset = k_offset; fused.v_offset = v_offset;
   fused.q_norm_w = q_norm_w; fused.k_norm_w = k_norm_w; fused.norm_dtype = norm_dtype; fused.eps = eps;
   fused.cos_sin = (const float2*)cos_sin;
+  fused.temp = xrt::query_temp(temp_coef, temp_every);
   fused.k_pool = write_kv ? (__nv_bfloat16*)k_pool : nullptr;
   fused.v_pool = write_kv ? (__nv_bfloat16*)v_pool : nullptr;
   return xrt::attention_decode_impl(out, part_o, part_ml, nullptr, k_pool, v_pool, n_blocks, tok_slot, tok_pos, block_table,

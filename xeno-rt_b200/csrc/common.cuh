@@ -114,6 +114,23 @@ struct KeyRange {
   }
 };
 
+// A temperature of the queries that grows with the logarithm of the position (every = 0: none): q at position p is
+// multiplied by 1 + coef * ln(floor((p + 1) / every) + 1), 32-bit, after its norm and rotation.
+struct QueryTemp {
+  float coef = 0.f;
+  int every = 0;
+  __device__ __forceinline__ float at(int pos) const {
+    return every > 0 ? fmaf(coef, logf((float)((pos + 1) / every + 1)), 1.0f) : 1.0f;
+  }
+};
+
+inline QueryTemp query_temp(float coef, int every) {
+  QueryTemp temp;
+  temp.coef = coef;
+  temp.every = every > 0 ? every : 0;
+  return temp;
+}
+
 inline KeyRange key_range(int window, int chunk) {
   KeyRange range;
   range.window = window;

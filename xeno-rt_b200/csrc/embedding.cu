@@ -1,7 +1,8 @@
 // Embedding gather: rows of the table to the 32-bit residual stream.
 // Restates crates/xrt-cuda/src/lib.rs:815-882 (embedding_kernel) of the reference, which writes
 // zeros for an id outside the table while its host wrapper refuses such ids (1217-1225); here the
-// kernel writes zeros and raises an error flag that the host reads.
+// kernel writes zeros and raises an error flag that the host reads.  With a table of positions the row of the token's
+// position is added to the (scaled) token row.
 #include "common.cuh"
 
 namespace xrt {
@@ -9,30 +10,37 @@ namespace xrt {
 template <typename TW>
 __global__ void embedding_kernel(float* __restrict__ out, const TW* __restrict__ table,
                                  const int* __restrict__ ids, int hidden, int vocab,
-                                 int* __restrict__ error_flag, float scale) {
+                                 int* __restrict__ error_flag, float scale, const TW* __restrict__ pos_table,
+                                 const int* __restrict__ positions, int n_positions) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const int id = ids[t];
-  const bool ok = id >= 0 && id < vocab;
+  const int at = pos_table != nullptr ? positions[t] : 0;
+  const bool ok = id >= 0 && id < vocab && (pos_table == nullptr || (at >= 0 && at < n_positions));
   if (!ok && threadIdx.x == 0 && error_flag != nullptr) atomicExch(error_flag, 1);
+  const TW* prow = pos_table != nullptr ? pos_table + (size_t)(ok ? at : 0) * hidden : nullptr;
   const TW* row = table + (size_t)(ok ? id : 0) * hidden;
   float* dst = out + (size_t)t * hidden;
-  for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = ok ? to_float(row[c]) * scale : 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x)
+    dst[c] = ok ? to_float(row[c]) * scale + (prow != nullptr ? to_float(prow[c]) : 0.f) : 0.f;
 }
 
 // 16 bytes of the table a thread and step (hidden a multiple of 8 for bfloat16, of 4 for float32)
 template <typename TW>
 __global__ void embedding_vec_kernel(float* __restrict__ out, const TW* __restrict__ table,
                                      const int* __restrict__ ids, int hidden, int vocab,
-                                     int* __restrict__ error_flag, float scale) {
+                                     int* __restrict__ error_flag, float scale, const TW* __restrict__ pos_table,
+                                     const int* __restrict__ positions, int n_positions) {
   constexpr int PER = 16 / (int)sizeof(TW);
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const int id = ids[t];
-  const bool ok = id >= 0 && id < vocab;
+  const int at = pos_table != nullptr ? positions[t] : 0;
+  const bool ok = id >= 0 && id < vocab && (pos_table == nullptr || (at >= 0 && at < n_positions));
   if (!ok && threadIdx.x == 0 && error_flag != nullptr) atomicExch(error_flag, 1);
+  const TW* prow = pos_table != nullptr ? pos_table + (size_t)(ok ? at : 0) * hidden : nullptr;
   const TW* row = table + (size_t)(ok ? id : 0) * hidden;
   float* dst = out + (size_t)t * hidden;
 #pragma unroll 4
@@ -42,6 +50,12 @@ __global__ void embedding_vec_kernel(float* __restrict__ out, const TW* __restri
     float f[PER];
 #pragma unroll
     for (int j = 0; j < PER; ++j) f[j] = ok ? to_float(vals[j]) * scale : 0.f;
+    if (prow != nullptr && ok) {
+      const uint4 praw = *reinterpret_cast<const uint4*>(prow + c);
+      const TW* pvals = reinterpret_cast<const TW*>(&praw);
+#pragma unroll
+      for (int j = 0; j < PER; ++j) f[j] += to_float(pvals[j]);
+    }
 #pragma unroll
     for (int j = 0; j < PER; j += 4) *reinterpret_cast<float4*>(dst + c + j) = make_float4(f[j], f[j + 1], f[j + 2], f[j + 3]);
   }
@@ -109,15 +123,16 @@ XRT_EXPORT int xrt_embedding_pair(float* out, const void* table, const void* pai
 }
 
 XRT_EXPORT int xrt_embedding(float* out, const void* table, const int* ids, int n_tokens, int hidden,
-                             int vocab, int table_dtype, int* error_flag, float scale, cudaStream_t stream) {
-  if (n_tokens < 0 || hidden <= 0 || vocab <= 0) return XRT_ERR_ARGUMENT;
+                             int vocab, int table_dtype, int* error_flag, float scale, const void* pos_table,
+                             const int* positions, int n_positions, cudaStream_t stream) {
+  if (n_tokens < 0 || hidden <= 0 || vocab <= 0 || (pos_table != nullptr && positions == nullptr)) return XRT_ERR_ARGUMENT;
   if (n_tokens == 0) return XRT_OK;
-  const bool vec = hidden % 8 == 0 && (((uintptr_t)out | (uintptr_t)table) & 15) == 0;
+  const bool vec = hidden % 8 == 0 && (((uintptr_t)out | (uintptr_t)table | (uintptr_t)pos_table) & 15) == 0;
   XRT_DISPATCH_DTYPE(table_dtype, TW, {
     if (vec)
-      xrt::launch_kernel(xrt::embedding_vec_kernel<TW>, dim3(n_tokens), dim3(128), 0, stream, out, (const TW*)table, ids, hidden, vocab, error_flag, scale);
+      xrt::launch_kernel(xrt::embedding_vec_kernel<TW>, dim3(n_tokens), dim3(128), 0, stream, out, (const TW*)table, ids, hidden, vocab, error_flag, scale, (const TW*)pos_table, positions, n_positions);
     else
-      xrt::launch_kernel(xrt::embedding_kernel<TW>, dim3(n_tokens), dim3(256), 0, stream, out, (const TW*)table, ids, hidden, vocab, error_flag, scale);
+      xrt::launch_kernel(xrt::embedding_kernel<TW>, dim3(n_tokens), dim3(256), 0, stream, out, (const TW*)table, ids, hidden, vocab, error_flag, scale, (const TW*)pos_table, positions, n_positions);
   });
   return xrt::launch_status();
 }

@@ -26,12 +26,14 @@ _F = ctypes.c_float
 _CODES = {torch.float32: 0, torch.bfloat16: 1}
 
 _SIGNATURES = {
-    "xrt_embedding": [_P, _P, _P, _I, _I, _I, _I, _P, _F, _P],
+    "xrt_embedding": [_P, _P, _P, _I, _I, _I, _I, _P, _F, _P, _P, _I, _P],
     "xrt_rmsnorm": [_P, _P, _P, _P, _I, _I, _F, _I, _I, _P],
     "xrt_layernorm": [_P, _P, _P, _P, _I, _I, _F, _I, _I, _P],
     "xrt_swiglu": [_P, _P, _I, _I, _I, _I, _I, _P, _P],
     "xrt_rotation_table": [_P, _P, _P, _P, _F, _I, _I, _P],
     "xrt_state_scan": [_P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
+    "xrt_head_scan": [_P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _P],
+    "xrt_stream_add": [_P, _P, ctypes.c_longlong, _I, _P, _P, _P, _P, _F, _F, _P, _P, _F, _I, _I, _I, _I, _P],
     "xrt_removal_gates": [_P, _I, _P, _P, _I, _P, _P, _I, _P, _I, _I, _I, _I, _F, _F, _P],
     "xrt_rmsnorm_shift": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _P],
     "xrt_add_row": [_P, _P, _I, _I, _I, _P],
@@ -51,7 +53,7 @@ _SIGNATURES = {
     "xrt_embedding_pair": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "xrt_layernorm_affine": [_P, _P, _P, _I, ctypes.c_longlong, _P, _P, _P, _I, _I, _F, _I, _P, _P, _P],
     "xrt_qkv_heads_write": [_P, _P, _P, _P, _I, _I, _I, _P, _I, _I, _F, _P, _P, _I, _I, _I, _P, _I, _I,
-                            _P, _I, _P, _I, _F, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+                            _P, _I, _P, _I, _F, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P],
     "xrt_rmsnorm_add": [_P, _P, ctypes.c_longlong, _I, _P, _P, _I, _I, _F, _I, _I, _P, _P, _F, _P, _P, _F, _P],
     "xrt_cast_rows": [_P, _P, ctypes.c_longlong, _I, _P],
     "xrt_latent_prepare": [_P, _P, _P, _I, _I, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
@@ -66,7 +68,7 @@ _SIGNATURES = {
     "xrt_scale_softcap": [_P, _I, _I, _F, _F, _P],
     "xrt_rope_table": [_P, _P, _P, _F, _I, _I, _P],
     "xrt_qk_rope_kv_write": [_P, _P, _P, _P, _I, _I, _I, _P, _P, _F, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I,
-                             _I, _I, _I, _I, _I, _P],
+                             _I, _I, _I, _I, _I, _F, _I, _P],
     "xrt_attention_reference": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _P, _I, _I, _I, _I, _P],
     "xrt_gemm_reference": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "xrt_gemm_stream": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
@@ -81,7 +83,7 @@ _SIGNATURES = {
     "xrt_attention_decode_fused": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _P, _I, _P, _I],
     "xrt_attention_decode": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _P, _I, _P, _I],
     "xrt_attention_decode_qkv": [_P, _P, _P, _P, _P, _I, _I, _I, _P, _P, _I, _F, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I,
-                                 _I, _I, _F, _I, _I, _I, _P, _P, _P, _I, _P, _I],
+                                 _I, _I, _F, _I, _I, _I, _P, _P, _P, _I, _P, _I, _F, _I],
     "xrt_attention_decode_scored": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _P, _I, _I, _I, _P],
     "xrt_attention_prefill": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _F, _F, _I, _F, _P, _I, _P],
     "xrt_attention_prefill_tcgen05": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _I, _I, _P],
@@ -257,15 +259,21 @@ def _check(status: int, what: str) -> None:
     raise KernelError(f"{what}: CUDA launch error {status}")
 
 
-def embedding(out, table, ids, error_flag, scale: float = 1.0) -> None:
-    """out[t, :] = table[ids[t], :] * scale as float32; raises error_flag[0] on an id outside the table."""
+def embedding(out, table, ids, error_flag, scale: float = 1.0, pos_table=None, positions=None) -> None:
+    """out[t, :] = table[ids[t], :] * scale as float32, plus pos_table[positions[t], :] where given (the table's dtype;
+    not scaled); raises error_flag[0] on an id or a position outside its table."""
     n, hidden = out.shape
     vocab = table.shape[0]
     if table.shape[1] != hidden or ids.numel() != n:
         raise KernelError("embedding: shapes do not fit")
+    if pos_table is not None and (pos_table.shape[1] != hidden or pos_table.dtype != table.dtype or positions is None
+                                  or positions.numel() != n):
+        raise KernelError("embedding: the table of positions does not fit")
     _check(_kernels().xrt_embedding(_ptr(out, "out", torch.float32), _ptr(table, "table"),
                                    _ptr(ids, "ids", torch.int32), n, hidden, vocab, _code(table.dtype),
-                                   _ptr(error_flag, "error_flag", torch.int32), float(scale), _stream()), "embedding")
+                                   _ptr(error_flag, "error_flag", torch.int32), float(scale), _ptr(pos_table, "pos_table"),
+                                   _ptr(positions if pos_table is not None else None, "positions", torch.int32),
+                                   pos_table.shape[0] if pos_table is not None else 0, _stream()), "embedding")
 
 
 def rmsnorm(out, x, weight, eps: float, rows=None) -> None:
@@ -354,8 +362,10 @@ def rope_table(cos_sin, positions, freq, scale: float) -> None:
 
 def qk_rope_kv_write(q_out, k_pool, v_pool, qkv, k_offset: int, v_offset: int, q_norm_w, k_norm_w, eps: float,
                      cos_sin, tok_slot, tok_pos, block_table, n_heads: int, n_kv_heads: int, head_dim: int,
-                     write_kv: bool = True, pairing: str = "split_half") -> None:
-    """Head norms, rotation, q output and cache write in one kernel; see rotary_kv.cu.  ``cos_sin``
+                     write_kv: bool = True, pairing: str = "split_half", q_temp=None) -> None:
+    """Head norms, rotation, q output and cache write in one kernel; see rotary_kv.cu.  ``q_temp`` = (coef, every) or
+    None: q at position p times 1 + coef * ln((p + 1) // every + 1).  ``v_offset`` may equal ``k_offset`` (the values
+    are the projected keys, before norm and rotation).  ``cos_sin``
     [T, rope_dim / 2, 2] rotates the first rope_dim dims of every head: pairs (i, i + rope_dim / 2)
     with ``pairing`` "split_half", pairs (2i, 2i + 1) with "interleaved"; the rest stays as it is."""
     if pairing not in ("split_half", "interleaved"):
@@ -380,7 +390,17 @@ def qk_rope_kv_write(q_out, k_pool, v_pool, qkv, k_offset: int, v_offset: int, q
         _ptr(tok_pos, "tok_pos", torch.int32), _ptr(block_table, "block_table", torch.int32),
         block_table.shape[1], n, n_heads, n_kv_heads, head_dim, 1 if write_kv else 0,
         1 if pairing == "interleaved" else 0, _code(norm_dtype),
-        _code(q_out.dtype), _code(cache_dtype), _stream()), "qk_rope_kv_write")
+        _code(q_out.dtype), _code(cache_dtype), *_temp(q_temp), _stream()), "qk_rope_kv_write")
+
+
+def _temp(q_temp) -> tuple:
+    """(coef, every) of a query temperature for the launchers; every 0: none."""
+    if q_temp is None:
+        return 0.0, 0
+    coef, every = q_temp
+    if int(every) < 1:
+        raise KernelError("a query temperature needs a positive number of positions a step")
+    return float(coef), int(every)
 
 
 def _sink_args(sink, n_heads: int) -> tuple:
@@ -720,11 +740,12 @@ def attention_decode_takes_qkv(n_heads: int, n_kv_heads: int, head_dim: int, rop
 def attention_decode_qkv(out, qkv, k_offset: int, v_offset: int, q_norm_w, k_norm_w, eps: float, cos_sin, k_pool, v_pool,
                          tok_slot, tok_pos, block_table, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                          window: int, chunk: int, n_splits: int, write_kv: bool = True, fused: bool = True,
-                         clusters: bool = True, sinks=None, mask_chunk: int = 0) -> None:
+                         clusters: bool = True, sinks=None, mask_chunk: int = 0, q_temp=None) -> None:
     """Decode attention straight from the 32-bit output of the q/k/v product: per-head norms, rotation,
     the newest key and value into the cache (unless ``write_kv`` is False) and attention over the cache
     in ONE kernel (csrc/attention_decode.cu).  ``qkv``: float32 [n, row] with q at 0, k at ``k_offset``,
-    v at ``v_offset``.  Check ``attention_decode_takes_qkv`` first; other sizes raise."""
+    v at ``v_offset`` (``k_offset`` too where the values are the projected keys); ``q_temp`` as in ``qk_rope_kv_write``.
+    Check ``attention_decode_takes_qkv`` first; other sizes raise."""
     n = qkv.shape[0]
     if out.shape != (n, n_heads * head_dim) or tok_slot.numel() != n or tok_pos.numel() != n:
         raise KernelError("attention_decode_qkv: shapes do not fit")
@@ -749,7 +770,8 @@ def attention_decode_qkv(out, qkv, k_offset: int, v_offset: int, q_norm_w, k_nor
         _ptr(v_pool, "v_pool", torch.bfloat16), k_pool.shape[0], _ptr(tok_slot, "tok_slot", torch.int32),
         _ptr(tok_pos, "tok_pos", torch.int32), _ptr(block_table, "block_table", torch.int32), block_table.shape[1], n,
         n_heads, n_kv_heads, head_dim, float(scale), int(window), int(chunk), int(n_splits), flag.data_ptr(), _stream(),
-        ctypes.byref(merged), 1 if clusters else 0, _sinks(sinks, n_heads), int(mask_chunk)), "attention_decode_qkv")
+        ctypes.byref(merged), 1 if clusters else 0, _sinks(sinks, n_heads), int(mask_chunk), *_temp(q_temp)),
+        "attention_decode_qkv")
     if n_splits > 1 and not merged.value and (
             not use_counters or n_splits > attention_decode_fused_max_splits(head_dim, n_heads // n_kv_heads)):
         add_launches(1)  # the combine kernel
@@ -921,6 +943,76 @@ def state_scan(out, q, k, v, decay, beta, state, cu_seqlens, seq_slot, n_heads: 
                                     2 if unit is not None else (1 if delta else 0), int(max_new),
                                     _stream()),
            "state_scan")
+
+
+def head_scan(out, q, k, v, state, cu_seqlens, seq_slot, n_heads: int, n_qk_heads: int, dim: int, vdim: int,
+              decay=None, decay_raw=None, a_log=None, dt_bias=None, beta=None, q_scale: float = 1.0, unit_eps=None,
+              silu: bool = False, max_new: int = 0) -> None:
+    """The scan of a matrix state with ONE decay g a head: S <- g S + k v^T, or with ``beta`` (raw values [T, n_heads],
+    sigmoid taken here) the delta rule u = sigmoid(beta) (v - (g S)^T k), S <- g S + k u^T; out = S^T q * q_scale after
+    the write.  g is ``decay`` (float32 [n_heads], constant) or exp(-exp(a_log) softplus(decay_raw + dt_bias)) of a
+    raw value a token and head.  ``silu``: q, k and v pass silu first; ``unit_eps``: q and k are then divided by
+    sqrt(sum(x^2) + unit_eps) a head.  q, k [T, n_qk_heads * dim], v [T, n_heads * vdim], rows may be slices of wider
+    rows, all float32; ``state`` float32 [slots, n_heads, vdim, dim] is read and left as the sequences' last state.
+    ``max_new`` (0: not known): the most tokens a sequence brings."""
+    n = out.shape[0]
+    if out.shape != (n, n_heads * vdim) or out.dtype != torch.float32 or not out.is_contiguous():
+        raise KernelError("head_scan: out must be float32 [T, heads * vdim]")
+    if state.dim() != 4 or tuple(state.shape[1:]) != (n_heads, vdim, dim) or state.dtype != torch.float32:
+        raise KernelError("head_scan: the state must be float32 [slots, heads, vdim, dim]")
+    if (decay is None) == (decay_raw is None):
+        raise KernelError("head_scan: a decay is either a constant a head or a raw value a token and head")
+    if any(t is not None and t.shape[0] != n for t in (q, k, v, decay_raw, beta)):
+        raise KernelError("head_scan: one row a token is needed")
+    per_head = (decay,) if decay is not None else (a_log, dt_bias)
+    if any(t is None or t.numel() != n_heads for t in per_head):
+        raise KernelError("head_scan: one number a head is needed for the decay")
+    n_seqs = seq_slot.numel()
+    if cu_seqlens.numel() != n_seqs + 1:
+        raise KernelError("head_scan: cu_seqlens must hold one entry more than seq_slot")
+    qp, qs = _columns(q, "q", n_qk_heads * dim)
+    kp, ks = _columns(k, "k", n_qk_heads * dim)
+    vp, vs = _columns(v, "v", n_heads * vdim)
+    dp, ds = _columns(decay_raw, "decay_raw", n_heads) if decay_raw is not None else (0, 0)
+    bp, bs = _columns(beta, "beta", n_heads) if beta is not None else (0, 0)
+    _check(_kernels().xrt_head_scan(
+        _ptr(out, "out"), qp, qs, kp, ks, vp, vs, dp, ds, _ptr(decay, "decay", torch.float32),
+        _ptr(a_log, "a_log", torch.float32), _ptr(dt_bias, "dt_bias", torch.float32), bp, bs, _ptr(state, "state"),
+        _ptr(cu_seqlens, "cu_seqlens", torch.int32), _ptr(seq_slot, "seq_slot", torch.int32), n_seqs, n_heads, n_qk_heads,
+        dim, vdim, float(q_scale), -1.0 if unit_eps is None else float(unit_eps), 1 if silu else 0, int(max_new), _stream()),
+        "head_scan")
+
+
+def stream_add(residual, y, factor: float = 1.0, rows=None, row_scales=None, scales=None, part_norms=None,
+               part_eps: float = 0.0, then=None) -> None:
+    """residual[t] += factor * sum_p s_p * part_p[t], 32-bit, the parts in index order.  ``y`` float32 [T, width] or
+    [parts, T, width]; or, with ``rows`` (int32 [T * parts]), [any, width] of which part p of token t is row
+    rows[t * parts + p].  s_p: ``row_scales`` (float32 [T, parts]), ``scales`` (float32 [parts]) or 1.  ``part_norms``
+    (float32 [parts, width], with ``part_eps``): every part's row is divided by its root mean square and multiplied by
+    that part's weight first.  ``then`` = (weight2, eps2, out2): out2 [T, width] receives RMSNorm(new residual) * weight2."""
+    n, width = residual.shape
+    if rows is not None:
+        if row_scales is None or row_scales.shape[0] != n or y.dim() != 2 or y.shape[1] != width:
+            raise KernelError("stream_add: gathered rows come as [any, width] with one scale a token and part")
+        parts = row_scales.shape[1]
+        if rows.numel() != n * parts:
+            raise KernelError("stream_add: one row index a token and part is needed")
+    else:
+        parts = y.shape[0] if y.dim() == 3 else 1
+        if tuple(y.shape[-2:]) != (n, width):
+            raise KernelError("stream_add: shapes do not fit")
+    if (row_scales is not None and tuple(row_scales.shape) != (n, parts)
+            or scales is not None and scales.numel() != parts or part_norms is not None and part_norms.numel() != parts * width):
+        raise KernelError("stream_add: the scales or the parts' norm weights do not fit")
+    then_w, then_eps, then_out = then if then is not None else (None, 0.0, None)
+    if then is not None and (tuple(then_out.shape) != (n, width) or then_w.numel() != width):
+        raise KernelError("stream_add: the norm that follows does not fit")
+    _check(_kernels().xrt_stream_add(
+        _ptr(residual, "residual", torch.float32), _ptr(y, "y", torch.float32), n * width, parts,
+        _ptr(rows, "rows", torch.int32), _ptr(row_scales, "row_scales", torch.float32), _ptr(scales, "scales", torch.float32),
+        _ptr(part_norms, "part_norms", torch.float32), float(part_eps), float(factor), _ptr(then_w, "then weight"),
+        _ptr(then_out, "then out"), float(then_eps), n, width, _code(then_w.dtype if then is not None else torch.float32),
+        _code(then_out.dtype if then is not None else torch.float32), _stream()), "stream_add")
 
 
 def short_conv(out, x, weight, state, cu_seqlens, seq_slot, max_new: int, act: str = "silu", bias=None, in_bias=None) -> None:
@@ -1241,7 +1333,7 @@ def qkv_heads_write(q_out, k_pool, v_pool, qkv, k_offset: int, v_offset: int, bi
                     eps: float, tok_slot, tok_pos, block_table, n_heads: int, n_kv_heads: int, head_dim: int,
                     v_keep=None, v_first=None, v_blend: float = 0.0, v_dim: int = 0, write_kv: bool = True,
                     q_norm_w=None, k_norm_w=None, whole_q: int = 0, whole_k: int = 0, cos_sin=None,
-                    pairing: str = "split_half", v_unit: bool = False) -> None:
+                    pairing: str = "split_half", v_unit: bool = False, q_temp=None) -> None:
     """``qk_rope_kv_write`` without rotation for layers that add a bias a column of the q/k/v row (float32, laid out as
     the row), divide q and k heads by their root mean square without a weight (over ``norm_dim`` dims where the heads
     are laid out wider), keep the values in 32-bit (``v_keep`` [T, kv heads * v_dim]) and / or cache
@@ -1249,7 +1341,8 @@ def qkv_heads_write(q_out, k_pool, v_pool, qkv, k_offset: int, v_offset: int, bi
     v_first hold the heads.  ``q_norm_w`` / ``k_norm_w`` with ``whole_q`` / ``whole_k`` > 0: an RMSNorm over the
     whole q (k) projection of a token, all heads at once, one weight a column of the projection as it is laid out, the
     number being the divisor of the mean of squares; ``cos_sin`` and ``pairing`` as in ``qk_rope_kv_write``.
-    ``v_unit``: every value head is divided by its root mean square over ``v_dim`` (``eps``, no weight) first."""
+    ``v_unit``: every value head is divided by its root mean square over ``v_dim`` (``eps``, no weight) first.
+    ``q_temp`` and ``v_offset`` as in ``qk_rope_kv_write``."""
     n = qkv.shape[0]
     if pairing not in ("split_half", "interleaved"):
         raise KernelError(f"qkv_heads_write: pairing {pairing!r} is not split_half or interleaved")
@@ -1288,7 +1381,7 @@ def qkv_heads_write(q_out, k_pool, v_pool, qkv, k_offset: int, v_offset: int, bi
         1 if pairing == "interleaved" else 0, kp, ks, fp, fs, float(v_blend), true_v, 1 if v_unit else 0,
         _ptr(tok_slot, "tok_slot", torch.int32), _ptr(tok_pos, "tok_pos", torch.int32),
         _ptr(block_table, "block_table", torch.int32), block_table.shape[1], n, n_heads, n_kv_heads, head_dim,
-        1 if write_kv else 0, _code(q_out.dtype), _code(cache_dtype), _stream()), "qkv_heads_write")
+        1 if write_kv else 0, _code(q_out.dtype), _code(cache_dtype), *_temp(q_temp), _stream()), "qkv_heads_write")
 
 
 def rmsnorm_add(residual, y, weight, eps: float, copy=None, factor: float = 1.0, part_scales=None, bias=None,

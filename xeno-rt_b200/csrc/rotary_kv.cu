@@ -94,7 +94,7 @@ __global__ void qk_rope_kv_write_kernel(
     const float2* __restrict__ cos_sin, int rope_half,
     const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
     const int* __restrict__ block_table, int max_blocks,
-    int n_heads, int n_kv_heads, int head_dim, int write_kv, int interleaved, const HeadExtras ex) {
+    int n_heads, int n_kv_heads, int head_dim, int write_kv, int interleaved, const QueryTemp temp, const HeadExtras ex) {
   extern __shared__ float staged[];  // [warps][head_dim]
   pdl_trigger();
   pdl_wait();
@@ -205,6 +205,11 @@ __global__ void qk_rope_kv_write_kernel(
   }
 
   if (kind == 0) {
+    if (temp.every > 0) {
+      const float f = temp.at(pos);
+#pragma unroll
+      for (int j = 0; j < MAX_PER_LANE; ++j) v[j] *= f;
+    }
     TQ* dst = q_out + (size_t)t * n_heads * head_dim + head * head_dim;
 #pragma unroll
     for (int j = 0; j < MAX_PER_LANE; ++j) {
@@ -248,7 +253,7 @@ qk_rope_kv_write_128_kernel(
     const float2* __restrict__ cos_sin, int rope_half,
     const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
     const int* __restrict__ block_table, int max_blocks,
-    int n_heads, int n_kv_heads, int write_kv) {
+    int n_heads, int n_kv_heads, int write_kv, const QueryTemp temp) {
   constexpr int HD = 128;
   pdl_trigger();
   // The step's arrays (slots, positions, block table) were written before the step began, and the norm
@@ -265,6 +270,7 @@ qk_rope_kv_write_128_kernel(
 #pragma unroll
     for (int j = 0; j < 4; ++j) { qn[j] = to_float(q_norm_w[4 * lane + j]); kn[j] = to_float(k_norm_w[4 * lane + j]); }
   }
+  const float q_factor = temp.at(pos);
   pdl_wait();
   // (cos, sin) of this lane's four pairs: dims 4 * (lane % 16) .. of the first half
   float c[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
@@ -323,6 +329,10 @@ qk_rope_kv_write_128_kernel(
         }
       }
       if (kind == 0) {
+        if (temp.every > 0) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[j] *= q_factor;
+        }
         store4_as(q_out + (size_t)t * n_heads * HD + head * HD + 4 * lane, v);
       } else if (block >= 0) {  // the host reserves blocks before the step; otherwise nothing to write into
         TC* pool = kind == 1 ? k_pool : v_pool;
@@ -358,14 +368,16 @@ XRT_EXPORT int xrt_rotation_table(float* cos_sin, const int* pos, const float* f
 
 // qkv: 32-bit rows of `row_stride` floats holding q at 0, k at k_offset, v at v_offset.
 // q_out: [n_tokens, n_heads * head_dim] in q_dtype.  k_pool / v_pool: the cache blocks of this
-// layer, [n_blocks, n_kv_heads, 64, head_dim] in cache_dtype.  Norm weights may be null (no head
+// layer, [n_blocks, n_kv_heads, 64, head_dim] in cache_dtype.  v_offset may equal k_offset: the values are then the
+// projected keys as they stand before norm and rotation.  Norm weights may be null (no head
 // norm) and share norm_dtype.  write_kv = 0 leaves the cache alone (a layer reading another's).
 static int qk_rope_kv_write(void* q_out, void* k_pool, void* v_pool, const float* qkv, int row_stride,
                             int k_offset, int v_offset, const void* q_norm_w, const void* k_norm_w,
                             float eps, const float* cos_sin, int rope_half, const int* tok_slot,
                             const int* tok_pos, const int* block_table, int max_blocks, int n_tokens,
                             int n_heads, int n_kv_heads, int head_dim, int write_kv, int interleaved,
-                            int norm_dtype, int q_dtype, int cache_dtype, const xrt::HeadExtras& ex, cudaStream_t stream) {
+                            int norm_dtype, int q_dtype, int cache_dtype, const xrt::QueryTemp& temp, const xrt::HeadExtras& ex,
+                            cudaStream_t stream) {
   const bool plain = ex.bias == nullptr && !ex.unit_norm && ex.norm_dim == 0 && ex.v_keep == nullptr && ex.v_first == nullptr &&
                      ex.whole_q == 0 && ex.whole_k == 0 && !ex.v_unit;
   if (n_tokens < 0 || n_heads <= 0 || n_kv_heads <= 0 || head_dim <= 0) return XRT_ERR_ARGUMENT;
@@ -382,7 +394,7 @@ static int qk_rope_kv_write(void* q_out, void* k_pool, void* v_pool, const float
           xrt::launch_kernel(xrt::qk_rope_kv_write_128_kernel<TN, TQ, TC>, dim3(n_tokens), dim3(256), 0, stream,
               (TQ*)q_out, (TC*)k_pool, (TC*)v_pool, qkv, row_stride, k_offset, v_offset, (const TN*)q_norm_w,
               (const TN*)k_norm_w, eps, (const float2*)cos_sin, rope_half, tok_slot, tok_pos, block_table,
-              max_blocks, n_heads, n_kv_heads, write_kv);
+              max_blocks, n_heads, n_kv_heads, write_kv, temp);
         });
       });
     });
@@ -398,7 +410,7 @@ static int qk_rope_kv_write(void* q_out, void* k_pool, void* v_pool, const float
         xrt::launch_kernel(xrt::qk_rope_kv_write_kernel<TN, TQ, TC, 8>, grid, dim3(warps * 32), smem, stream,
             (TQ*)q_out, (TC*)k_pool, (TC*)v_pool, qkv, row_stride, k_offset, v_offset, (const TN*)q_norm_w,
             (const TN*)k_norm_w, eps, (const float2*)cos_sin, rope_half, tok_slot, tok_pos, block_table,
-            max_blocks, n_heads, n_kv_heads, head_dim, write_kv, interleaved, ex);
+            max_blocks, n_heads, n_kv_heads, head_dim, write_kv, interleaved, temp, ex);
       });
     });
   });
@@ -410,10 +422,12 @@ XRT_EXPORT int xrt_qk_rope_kv_write(void* q_out, void* k_pool, void* v_pool, con
                                     float eps, const float* cos_sin, int rope_half, const int* tok_slot,
                                     const int* tok_pos, const int* block_table, int max_blocks, int n_tokens,
                                     int n_heads, int n_kv_heads, int head_dim, int write_kv, int interleaved,
-                                    int norm_dtype, int q_dtype, int cache_dtype, cudaStream_t stream) {
+                                    int norm_dtype, int q_dtype, int cache_dtype, float temp_coef, int temp_every,
+                                    cudaStream_t stream) {
   return qk_rope_kv_write(q_out, k_pool, v_pool, qkv, row_stride, k_offset, v_offset, q_norm_w, k_norm_w, eps, cos_sin,
                           rope_half, tok_slot, tok_pos, block_table, max_blocks, n_tokens, n_heads, n_kv_heads, head_dim,
-                          write_kv, interleaved, norm_dtype, q_dtype, cache_dtype, xrt::HeadExtras(), stream);
+                          write_kv, interleaved, norm_dtype, q_dtype, cache_dtype, xrt::query_temp(temp_coef, temp_every),
+                          xrt::HeadExtras(), stream);
 }
 
 // The same with a bias a column, weightless unit norms of q and k, norms over the whole projection, and values that
@@ -427,7 +441,7 @@ XRT_EXPORT int xrt_qkv_heads_write(void* q_out, void* k_pool, void* v_pool, cons
                                    float v_blend, int v_dim, int v_unit, const int* tok_slot, const int* tok_pos,
                                    const int* block_table,
                                    int max_blocks, int n_tokens, int n_heads, int n_kv_heads, int head_dim, int write_kv,
-                                   int q_dtype, int cache_dtype, cudaStream_t stream) {
+                                   int q_dtype, int cache_dtype, float temp_coef, int temp_every, cudaStream_t stream) {
   xrt::HeadExtras ex;
   ex.v_unit = v_unit;
   ex.bias = bias;
@@ -443,5 +457,5 @@ XRT_EXPORT int xrt_qkv_heads_write(void* q_out, void* k_pool, void* v_pool, cons
   ex.whole_k = whole_k;
   return qk_rope_kv_write(q_out, k_pool, v_pool, qkv, row_stride, k_offset, v_offset, q_norm_w, k_norm_w, eps, cos_sin,
                           rope_half, tok_slot, tok_pos, block_table, max_blocks, n_tokens, n_heads, n_kv_heads, head_dim,
-                          write_kv, interleaved, norm_dtype, q_dtype, cache_dtype, ex, stream);
+                          write_kv, interleaved, norm_dtype, q_dtype, cache_dtype, xrt::query_temp(temp_coef, temp_every), ex, stream);
 }

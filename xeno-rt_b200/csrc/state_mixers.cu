@@ -19,15 +19,9 @@
 //
 // A sequence is a row of the step's cu_seqlens / seq_slot arrays; a row with slot -1 or no tokens is
 // skipped, so padding rows of a captured step leave every state alone.
-#include "common.cuh"
+#include "recurrence.cuh"
 
 namespace xrt {
-
-__device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float softplusf_(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float activate(float z, int act) {  // 0 none, 1 silu, 2 sigmoid, 3 tanh
-  return act == 1 ? z * sigmoidf_(z) : (act == 2 ? sigmoidf_(z) : (act == 3 ? tanhf(z) : z));
-}
 
 // ------------------------------------------------------------------------------------------ the scan
 // One block: one sequence, one head, COLS value columns.  A column's state S[:, j] (dim rows) is held
@@ -39,15 +33,6 @@ __device__ __forceinline__ float activate(float z, int act) {  // 0 none, 1 silu
 // worked on.  A lane's rows are every PARTS-th group of four (lane p holds rows 4 (i PARTS + p) .. + 3), so
 // that the lanes of a column read neighbouring 16 bytes at a time: whole lines of the state in global
 // memory, different banks of shared memory.  Sums over a lane's rows run as two chains.
-template <int BYTES>
-__device__ __forceinline__ void cp_async(float* smem, const float* global) {
-  const unsigned dst = (unsigned)__cvta_generic_to_shared(smem);
-  if (BYTES == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(global) : "memory");
-  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(global) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
 struct ScanArgs {
   float* out;
   const float *q, *k, *v, *decay, *beta;

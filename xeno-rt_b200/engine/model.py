@@ -163,6 +163,8 @@ class Model:
         if hasattr(self.embedding, "state_need"):
             x = x0 = self.embedding.forward(ctx.token_ids, self.error_flag, ctx=ctx,
                                             state=cache.sequence_state["embedding"])
+        elif getattr(self.embedding, "takes_context", False):  # an embedding that looks at the tokens' positions
+            x = x0 = self.embedding.forward(ctx.token_ids, self.error_flag, ctx=ctx)
         else:
             x = x0 = self.embedding.forward(ctx.token_ids, self.error_flag)
         if self.stream_parts and self.spec.schedule[0].before is None:

@@ -6,5 +6,6 @@ from . import guzuvik  # registers Guzuvik
 from . import zogevik  # registers Zogevik
 from . import sofunex  # registers Sofunex
 from . import fadutar  # registers Fadutar
+from . import zivovik  # registers Zivovik
 
-__all__ = ["llama", "givopel", "guzuvik", "zogevik", "sofunex", "fadutar"]
+__all__ = ["llama", "givopel", "guzuvik", "zogevik", "sofunex", "fadutar", "zivovik"]

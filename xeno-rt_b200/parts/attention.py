@@ -72,7 +72,9 @@ class GroupedQueryAttention:
     ``k_conv``, ``v_conv`` [channels, taps], right after the product and its bias, before norms and rotation; the
     last taps - 1 rows of the product are state of the sequence, so the part then asks for a ``StateNeed`` beside
     its keys), ``v_norm`` = "unit" (every value head is divided by its root mean square, ``eps``, no weight, before it
-    is cached), ``o_bias`` (the output product has a bias ``o_bias`` [width]).
+    is cached), ``o_bias`` (the output product has a bias ``o_bias`` [width]), ``tied_values`` (the values are the keys as
+    projected, before norm and rotation: no ``v`` tensor; the value size is head_dim), ``q_temp`` ({"coef", "every"}: the
+    queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1) after norm and rotation).
     weights: ``q`` [n_heads*head_dim, width], ``k`` [n_kv_heads*head_dim, width], ``v``
     [n_kv_heads*v_head_dim, width], ``o`` [width, n_heads*v_head_dim], with qk_norm ``q_norm``,
     ``k_norm`` [head_dim], with a gate ``g`` [n_heads*v_head_dim, width].
@@ -96,6 +98,8 @@ class GroupedQueryAttention:
         hd, vd, size = cls._sizes(params)
         if hd != size or vd != size or not params.get("own_kv", True):
             return {}  # the part lays the heads out itself
+        if params.get("tied_values"):
+            return {"qkg": ("q", "k", "g")} if params.get("gate") else {"qk": ("q", "k")}
         return {"qkvg": ("q", "k", "v", "g")} if params.get("gate") else {"qkv": ("q", "k", "v")}
 
     @staticmethod
@@ -119,6 +123,8 @@ class GroupedQueryAttention:
         if not params.get("own_kv", True):
             for role in ("k", "v", "k_norm"):
                 shapes.pop(role, None)
+        if params.get("tied_values"):
+            shapes.pop("v", None)
         if params.get("gate"):
             shapes["g"] = ((nh if params["gate"] == "sigmoid_head" else nh * vd, d), "matrix")
         if params.get("bias"):
@@ -153,6 +159,13 @@ class GroupedQueryAttention:
         self.chunk = int(params.get("chunk") or 0)
         if not self.own_kv and (params.get("bias") or params.get("value_blend")):
             raise Unsupported("a layer without keys and values of its own cannot have their biases or blend them")
+        self.tied_values = bool(params.get("tied_values"))
+        if self.tied_values and (true_vdim != true_dim or params.get("bias") or params.get("conv")):
+            raise Unsupported("values that are the projected keys have the keys' size, and no biases or convolutions")
+        temp = params.get("q_temp")
+        self.q_temp = (float(temp["coef"]), int(temp["every"])) if temp else None
+        if self.q_temp is not None and self.q_temp[1] < 1:
+            raise ConfigError(f"q_temp.every {self.q_temp[1]} must be at least 1")
         self.keep_first = int(params.get("keep_first") or 0) if self.window else 0
         self.softcap = float(params.get("softcap") or 0.0)
         self.distance_rate = float(params.get("distance_rate") or 0.0)
@@ -168,13 +181,14 @@ class GroupedQueryAttention:
         self.q_width = self.n_heads * self.head_dim
         self.kv_width = self.n_kv_heads * self.head_dim
         # one fused weight for the products that read the mixer's input; the reference fuses only their dispatch (447-486)
-        self.w_qkv = weights.get("qkvg" if self.gate else "qkv")
+        self.w_qkv = weights.get(("qk" if self.tied_values else "qkv") + ("g" if self.gate else ""))
         self.w_o = weights["o"]
         if self.w_qkv is None:  # tensors that came one by one, or heads that are laid out at another size
             pieces = [_pad_rows(weights["q"], self.n_heads, true_dim, self.head_dim)]
             if self.own_kv:
-                pieces += [_pad_rows(weights["k"], self.n_kv_heads, true_dim, self.head_dim),
-                           _pad_rows(weights["v"], self.n_kv_heads, true_vdim, self.head_dim)]
+                pieces.append(_pad_rows(weights["k"], self.n_kv_heads, true_dim, self.head_dim))
+                if not self.tied_values:
+                    pieces.append(_pad_rows(weights["v"], self.n_kv_heads, true_vdim, self.head_dim))
             if self.gate == "sigmoid_head":
                 pieces.append(weights["g"])
             elif self.gate:
@@ -183,7 +197,8 @@ class GroupedQueryAttention:
             if true_vdim != self.head_dim:
                 self.w_o = _pad_columns(weights["o"], self.n_heads, true_vdim, self.head_dim)
         self.w_q = self.w_qkv[: self.q_width]
-        self.gate_offset = self.q_width + 2 * self.kv_width
+        self.v_offset = self.q_width + (0 if self.tied_values else self.kv_width)
+        self.gate_offset = self.v_offset + self.kv_width
         weighted = params.get("qk_norm") and not self.unit_norm
         self.q_norm = weights.get("q_norm") if weighted else None
         self.k_norm = weights.get("k_norm") if weighted else None
@@ -221,6 +236,11 @@ class GroupedQueryAttention:
         # ops.qkv_heads_write and attend with the kernels that take the score options
         self.plain_heads = (self.bias is None and not self.unit_norm and not self.whole_norm and not self.value_blend
                             and true_dim == self.head_dim and not self.taps and not self.v_unit)
+        if (self.unit_norm and true_dim == self.head_dim and self.bias is None and not self.value_blend and not self.taps
+                and not self.v_unit):
+            # a norm without a weight is one whose weight is ones: the kernels that fold norms in take it as that
+            self.q_norm = self.k_norm = torch.ones(self.head_dim, dtype=torch.float32, device=device)
+            self.plain_heads = True
         self.plain_scores = not (self.keep_first or self.softcap or self.distance_rate)
         position = params.get("position") or {"kind": "none", "params": {}}
         self.position = part_class("position", position["kind"])(position.get("params", {}), {}, dtype, device)
@@ -293,17 +313,18 @@ class GroupedQueryAttention:
         attended = (torch.zeros if padded else torch.empty)((n, self.q_width), dtype=self.act_dtype, device=h.device)
         if self.dtype is DType.BF16 and self.plain_heads and self.plain_scores:
             from . import attention_bf16
-            if attention_bf16.decode_from_qkv(attended, qkv, self.q_width, self.q_width + self.kv_width, self.q_norm,
+            if attention_bf16.decode_from_qkv(attended, qkv, self.q_width, self.v_offset, self.q_norm,
                                               self.k_norm, self.eps, cos_sin, pairing, ctx, store, self.n_heads,
                                               self.n_kv_heads, self.head_dim, self.scale, window, owns_cache, self.sinks,
-                                              self.chunk):
+                                              self.chunk, self.q_temp):
                 qkv = None
         if qkv is not None:
             q = torch.empty((n, self.q_width), dtype=self.act_dtype, device=h.device)
             if self.plain_heads:
-                ops.qk_rope_kv_write(q, store.k, store.v, qkv, self.q_width, self.q_width + self.kv_width, self.q_norm,
+                ops.qk_rope_kv_write(q, store.k, store.v, qkv, self.q_width, self.v_offset, self.q_norm,
                                      self.k_norm, self.eps, cos_sin, ctx.tok_slot, ctx.tok_pos, store.block_table,
-                                     self.n_heads, self.n_kv_heads, self.head_dim, write_kv=owns_cache, pairing=pairing)
+                                     self.n_heads, self.n_kv_heads, self.head_dim, write_kv=owns_cache, pairing=pairing,
+                                     q_temp=self.q_temp)
             else:
                 v_keep = v_first = None
                 if self.value_blend and owns_cache:
@@ -313,14 +334,14 @@ class GroupedQueryAttention:
                     if v_first is None:  # the first layer of this name in the step: its values are the ones blended in
                         v_keep = torch.zeros((n, self.n_kv_heads * self.true_vdim), dtype=torch.float32, device=h.device)
                         ctx.shared[("value_blend", self.value_blend)] = v_keep
-                ops.qkv_heads_write(q, store.k, store.v, qkv, self.q_width, self.q_width + self.kv_width, bias,
+                ops.qkv_heads_write(q, store.k, store.v, qkv, self.q_width, self.v_offset, bias,
                                     self.unit_norm, self.true_dim, self.eps, ctx.tok_slot, ctx.tok_pos, store.block_table,
                                     self.n_heads, self.n_kv_heads, self.head_dim, v_keep=v_keep, v_first=v_first,
                                     v_blend=self.blend if v_first is not None else 0.0, v_dim=self.true_vdim,
                                     write_kv=owns_cache, q_norm_w=self.q_norm, k_norm_w=self.k_norm if owns_cache else None,
                                     whole_q=self.n_heads * self.true_dim if self.whole_norm else 0,
                                     whole_k=self.n_kv_heads * self.true_dim if self.whole_norm else 0,
-                                    cos_sin=cos_sin, pairing=pairing, v_unit=self.v_unit)
+                                    cos_sin=cos_sin, pairing=pairing, v_unit=self.v_unit, q_temp=self.q_temp)
             self.attend(attended, q, ctx, store)
         if self.gate == "sigmoid_head":
             ops.gate_mul(attended, projected[:, self.gate_offset:], "sigmoid", group=self.head_dim)

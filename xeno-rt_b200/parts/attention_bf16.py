@@ -74,7 +74,7 @@ def _decode_split_of(ctx, n_kv_heads: int, device, window: int = 0):
 
 
 def decode_from_qkv(out, qkv, k_offset, v_offset, q_norm, k_norm, eps, cos_sin, pairing, ctx, store, n_heads, n_kv_heads,
-                    head_dim, scale, window, write_kv, sinks=None, mask_chunk=0) -> bool:
+                    head_dim, scale, window, write_kv, sinks=None, mask_chunk=0, q_temp=None) -> bool:
     """A decode step's attention straight from the q/k/v product's output: the kernel does the head norms,
     the rotation and the cache write itself (one kernel and one boundary less a layer).  False where that
     kernel does not take the case; the caller then runs the rotation kernel and ``run``."""
@@ -86,7 +86,8 @@ def decode_from_qkv(out, qkv, k_offset, v_offset, q_norm, k_norm, eps, cos_sin, 
     fused = ctx.n_tokens * n_kv_heads <= FUSED_COMBINE_MAX
     ops.attention_decode_qkv(out, qkv, k_offset, v_offset, q_norm, k_norm, eps, cos_sin, store.k, store.v, ctx.tok_slot,
                              ctx.tok_pos, store.block_table, n_heads, n_kv_heads, head_dim, scale, window, chunk, n_splits,
-                             write_kv=write_kv, fused=fused, clusters=clusters, sinks=sinks, mask_chunk=mask_chunk)
+                             write_kv=write_kv, fused=fused, clusters=clusters, sinks=sinks, mask_chunk=mask_chunk,
+                             q_temp=q_temp)
     return True
 
 

@@ -103,6 +103,32 @@ def sandwich_residual(parts: LayerParts, x, ctx, stores, owns_cache: bool) -> No
         ctx.pending = ReadyNorm(following, h)
 
 
+def added_residual(parts: LayerParts, x, ctx, stores, owns_cache: bool) -> None:
+    """x += mixer(norm(x)); x += feed_forward(norm(x)) with a part of role ``add`` that says how a result enters the stream
+    (times a number, say).  The layer's parts are ``mixer_norm``, ``mixer``, ``mixer_add`` and, if it has a
+    feed-forward, ``ffn_norm``, ``ffn``, ``ffn_add``.  The mixer hands its result back (``mix``), the feed-forward too
+    (``apply_rows`` where it has that, else ``apply``), and the ``add`` part that takes it also computes the norm that
+    the next sublayer begins with (its own feed-forward's, or the first norm of the layer that runs next, left in
+    ``ctx.pending``)."""
+    ready = ctx.take_pending(parts.mixer_norm)
+    after = ctx.shared.get("next_layer")  # (first norm, the part that takes it, ..) of the layer that runs next, or None
+    following_layer = after[0] if after is not None and not (len(after) > 2 and "mixer_shift" in after[2]) else None
+    h = ready.value if isinstance(ready, ReadyNorm) else parts.mixer_norm.forward(x)
+    has_ffn = "ffn" in parts
+    following = parts.ffn_norm if has_ffn else following_layer
+    h = parts.mixer_add.add_into(x, parts.mixer.mix(h, ctx, stores.get("mixer"), owns_cache), then=following)
+    ctx.then_norm = ctx.pending = None
+    if has_ffn:
+        if h is None:
+            h = parts.ffn_norm.forward(x)
+        following = following_layer
+        give = getattr(parts.ffn, "apply_rows", parts.ffn.apply)
+        h = parts.ffn_add.add_into(x, give(h, ctx), then=following)
+        ctx.then_norm = ctx.pending = None
+    if h is not None:
+        ctx.pending = ReadyNorm(following, h)
+
+
 def postnorm_residual(parts: LayerParts, x, ctx, stores, owns_cache: bool) -> None:
     """x += norm(mixer(x)); x += norm(feed_forward(x)): the sublayers read the residual stream itself and only what
     they give is normed.  The layer's parts are ``mixer``, ``mixer_post`` and, if it has a feed-forward, ``ffn`` and
@@ -150,6 +176,8 @@ class ReadyNorm:
 
 
 sandwich_residual.first_norm = lambda parts: (parts.mixer_norm, parts.mixer, parts)
+added_residual.first_norm = lambda parts: (parts.mixer_norm, parts.mixer, parts)
+register_part("arrangement", "added_residual", added_residual)
 register_part("arrangement", "parallel_residual", parallel_residual)
 register_part("arrangement", "sandwich_residual", sandwich_residual)
 

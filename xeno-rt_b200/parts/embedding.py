@@ -9,24 +9,32 @@ from .registry import register_part
 
 
 class TokenEmbedding:
-    """x = E[token], no scaling (crates/xrt-models/src/llama.rs:1042-1055); with ``scale`` x = E[token] * scale (32-bit).
-    params: ``vocab_size``, ``width``, optional ``scale``.  weights: ``weight`` [vocab, width]."""
+    """x = E[token], no scaling (crates/xrt-models/src/llama.rs:1042-1055); with ``scale`` x = E[token] * scale (32-bit);
+    with ``positions`` (a number) a learned row a position is added, x = E[token] * scale + P[position].
+    params: ``vocab_size``, ``width``, optional ``scale``, ``positions``.  weights: ``weight`` [vocab, width], with
+    ``positions`` also ``positions`` [positions, width]."""
 
     graph_safe = True
 
     @classmethod
     def weight_shapes(cls, params):
-        return {"weight": ((params["vocab_size"], params["width"]), "matrix")}
+        shapes = {"weight": ((params["vocab_size"], params["width"]), "matrix")}
+        if params.get("positions"):
+            shapes["positions"] = ((int(params["positions"]), params["width"]), "matrix")
+        return shapes
 
     def __init__(self, params, weights, dtype, device):
         self.vocab_size = int(params["vocab_size"])
         self.width = int(params["width"])
         self.weight = weights["weight"]
         self.scale = float(params.get("scale") or 1.0)
+        self.positions = weights["positions"] if params.get("positions") else None
+        self.takes_context = self.positions is not None
 
-    def forward(self, token_ids, error_flag):
+    def forward(self, token_ids, error_flag, ctx=None):
         out = torch.empty((token_ids.numel(), self.width), dtype=torch.float32, device=token_ids.device)
-        ops.embedding(out, self.weight, token_ids, error_flag, self.scale)
+        ops.embedding(out, self.weight, token_ids, error_flag, self.scale, self.positions,
+                      ctx.tok_pos if self.positions is not None else None)
         return out
 
 

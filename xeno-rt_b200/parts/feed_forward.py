@@ -249,7 +249,12 @@ class RoutedExperts:
 
     GROUPED_FROM = 4  # (token, choice) pairs an expert from which a step's rows are sorted by expert
 
-    def apply(self, h, ctx):
+    def apply_rows(self, h, ctx):
+        """The same for a caller that takes ``WeightedParts`` of any form: where a step's rows are sorted by expert, the
+        experts' results stay where they lie and whoever adds them up gathers them (not with a shared expert)."""
+        return self.apply(h, ctx, gathered=self.shared is None)
+
+    def apply(self, h, ctx, gathered: bool = False):
         """The chosen experts' weighted results, float32 [top, T, width]; their sum in index order is the result.
         A step of few tokens runs every (token, choice) pair by itself, streaming that expert's matrices.  A step of
         many tokens (prompts, and decode steps of many sequences) sorts its rows by expert; in bfloat16 two launches
@@ -258,16 +263,18 @@ class RoutedExperts:
         once (prompts only)."""
         n = h.shape[0]
         ids, weights = self.route(h)
-        whole = torch.empty((self.top + (1 if self.shared else 0), n, self.width), dtype=torch.float32, device=h.device)
-        out = whole[:self.top]
-        if self.shared:
-            self.shared.apply(h, ctx, out=whole[self.top])
         pairs = n * self.top
         one_launch = h.dtype == torch.bfloat16 and self.width % 8 == 0 and self.inner % 8 == 0
         fixed_shapes = getattr(ctx, "captured", False) or ctx.all_single  # no read-back inside such a step
-        if pairs < self.GROUPED_FROM * self.experts or (fixed_shapes and not one_launch):
+        by_pair = pairs < self.GROUPED_FROM * self.experts or (fixed_shapes and not one_launch)
+        if by_pair or not gathered:
+            whole = torch.empty((self.top + (1 if self.shared else 0), n, self.width), dtype=torch.float32, device=h.device)
+            out = whole[:self.top]
+        if self.shared:
+            self.shared.apply(h, ctx, out=whole[self.top])
+        if by_pair:
             ops.moe_experts(out, h, self.w_in, self.w_out, ids, weights, self.inner, self.limit, self.alpha, act=self.act)
-            return whole
+            return WeightedParts(whole) if gathered else whole
         offsets = torch.empty((self.experts + 1,), dtype=torch.int32, device=h.device)
         pos = torch.empty((pairs,), dtype=torch.int32, device=h.device)
         row_token = torch.empty((pairs,), dtype=torch.int32, device=h.device)
@@ -292,6 +299,8 @@ class RoutedExperts:
                     gate_up = linear(rows[lo:hi], self.w_in[e * first:(e + 1) * first], out_dtype=torch.float32)
                     ops.moe_activation(act[lo:hi], gate_up, self.limit, self.alpha, kind=self.act)
                     linear(act[lo:hi], self.w_out[e * self.width:(e + 1) * self.width], accumulate_into=y[lo:hi])
+        if gathered:
+            return WeightedParts(y, rows=pos, row_scales=weights)
         ops.moe_combine(out, y, pos, weights)
         return whole
 

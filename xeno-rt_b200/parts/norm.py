@@ -6,7 +6,7 @@ from dataclasses import dataclass
 
 import torch
 
-from ..core import torch_dtype
+from ..core import ConfigError, torch_dtype
 from ..csrc import ops
 from .registry import register_part
 
@@ -43,10 +43,17 @@ class WeightedParts:
     """A sublayer's result that is still in parts: ``parts`` float32 [n, T, width], their sum sum_p scales[p] *
     parts[p] + bias being the result (``scales`` float32 [n] on the device or None for ones, ``bias`` float32 [width] or
     None; a result in one piece may be [T, width]).  The
-    norm that follows the sublayer adds them up in its own pass over the row."""
+    norm that follows the sublayer adds them up in its own pass over the row.
+    Two more forms, which only ``parts/stream_add.py:ScaledAdd`` takes: ``norms`` (float32 [n, width], with ``eps``): part
+    p counts as RMSNorm(parts[p]) * norms[p]; ``rows`` and ``row_scales`` (int32 [T * n], float32 [T, n]): ``parts`` is
+    [any, width] and part p of token t is its row rows[t * n + p] times row_scales[t, p] (experts' results where they lie)."""
     parts: torch.Tensor
     scales: torch.Tensor | None = None
     bias: torch.Tensor | None = None
+    norms: torch.Tensor | None = None
+    eps: float = 0.0
+    rows: torch.Tensor | None = None
+    row_scales: torch.Tensor | None = None
 
 
 class RMSNorm:
@@ -89,6 +96,8 @@ class RMSNorm:
         weight has this one's dtype; its result over the new residual is returned, computed in the same pass (else None)."""
         scales = bias = None
         if isinstance(y, WeightedParts):
+            if y.norms is not None or y.rows is not None:
+                raise ConfigError("a norm after a sublayer takes parts that are neither normed one by one nor gathered")
             y, scales, bias = y.parts, y.scales, y.bias
         if y.dim() == 3 and y.shape[0] == 1 and scales is None:
             y = y[0]

@@ -21,6 +21,8 @@ stream          ``forward(x, x0, ctx) -> x``: a step on the residual stream betw
                 the embedding gave.  It may return a new tensor.  A ``SchedulePlace`` names it in ``before``.
 shift           ``cache_need() -> StateNeed`` and ``forward(x, norm, ctx, store, owns_cache) -> h``: the norm of the
                 stream blended with what it was for the token before (kept for every sequence).
+add             ``add_into(x, y, then=None) -> normed | None``: a sublayer's result ``y`` enters the stream ``x`` in place;
+                ``then`` is the norm part that the next sublayer begins with, whose result may be computed on the way.
 A mixer may also have ``mix(h, ctx, store, owns_cache) -> float32 [T, D]``: its result handed back instead
 of added, for a mixer that is made of other mixers.
 A part class may set ``graph_safe = True`` to say that its ``forward`` only launches device work
@@ -38,7 +40,8 @@ from __future__ import annotations
 
 from ..core import ConfigError
 
-ROLES = ("norm", "mixer", "feed_forward", "position", "embedding", "lm_head", "arrangement", "stream", "shift")
+ROLES = ("norm", "mixer", "feed_forward", "position", "embedding", "lm_head", "arrangement", "stream", "shift",
+         "add")
 _REGISTRY: dict[str, dict[str, object]] = {role: {} for role in ROLES}
 
 

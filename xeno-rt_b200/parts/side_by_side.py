@@ -1,5 +1,6 @@
 """A mixer made of several mixers that read the same input side by side: each one's result is RMS-normed
-over the model width with a weight of its own, and the mean of those is the mixer's result.
+over the model width with a weight of its own, and the mean of those is the mixer's result.  ``forward`` adds it
+into the stream; ``mix`` hands it back as parts to be normed and averaged (a ``WeightedParts`` with ``norms``).
 
 params: ``width``, ``eps``, ``branches``: a list of ``{"name", "kind", "params"}`` naming registered mixers
 (each must offer ``mix``).  weights: for branch ``name`` the branch's own tensors under ``<name>.<role>``
@@ -58,7 +59,10 @@ class SideBySideMixer:
             self.branches.append(branch_cls(branch_params, own, dtype, device))
             if self.combine != "weighted":
                 self.out_weights.append(weights[f"{name}.out"].to(torch.float32).contiguous())
-        self.bias = None
+        self.bias = self.norms = None
+        if self.combine == "normed_mean" and self.out_weights:
+            self.norms = torch.stack(self.out_weights).contiguous()
+            self.scales = torch.full((len(self.branches),), 1.0 / len(self.branches), dtype=torch.float32, device=device)
         if self.combine == "weighted":
             factors = [float(b["scale"]) for b in params["branches"]]
             self.scales = torch.tensor(factors, dtype=torch.float32, device=device)
@@ -75,18 +79,16 @@ class SideBySideMixer:
         return [b.cache_need() for b in self.branches]
 
     def mix(self, h, ctx, store, owns_cache=True):
-        """The branches' results as parts with their factors (``combine`` "weighted" only)."""
+        """The branches' results as parts with their factors (and, for ``combine`` "normed_mean", their norms)."""
         from .norm import WeightedParts
-        if self.combine != "weighted":
-            raise ConfigError("side-by-side mixers whose results are normed and averaged add into the stream themselves")
         ctx.then_norm = None
         parts = torch.empty((len(self.branches), h.shape[0], self.width), dtype=torch.float32, device=h.device)
         for i, (branch, branch_store) in enumerate(zip(self.branches, store)):
-            if getattr(branch, "o_bias", None) is not None:
+            if self.combine == "weighted" and getattr(branch, "o_bias", None) is not None:
                 branch.mix(h, ctx, branch_store, owns_cache, out=parts[i], leave_bias=True)
             else:
                 branch.mix(h, ctx, branch_store, owns_cache, out=parts[i])
-        return WeightedParts(parts, self.scales, self.bias)
+        return WeightedParts(parts, self.scales, self.bias, norms=self.norms, eps=self.eps)
 
     def forward(self, h, residual, ctx, store, owns_cache=True):
         ctx.then_norm = None

@@ -1,6 +1,8 @@
-"""Mixers that keep a matrix state per head instead of keys and values: gated linear attention, the gated delta
+"""Mixers that keep a matrix state per head instead of keys and values: gated linear attention, linear attention
+with a constant decay a head, the gated delta
 rule, and a delta rule with a decay and a removal rate per key channel (``DecayRemovalRule``, whose recurrence is in
-its own text).  All run the same scan kernel (csrc/state_mixers.cu) over the tokens of a step,
+its own text).  All run a scan over the tokens of a step (csrc/state_mixers.cu; where the decay is one number a head
+csrc/head_scan.cu),
 
     S_t = diag(a_t) S_(t-1) + k_t u_t^T,        o_t = S_t^T q_t,
 
@@ -108,6 +110,9 @@ class GatedDeltaRule(_StateMixer):
     head; decay a = exp(-exp(A_log[head]) * softplus(W_a2 (W_a1 h) + dt_bias)) per head and key channel; scan with
     the delta rule; every head's o divided by its root mean square (eps), times the shared weight ``norm``, times
     sigmoid(W_g2 (W_g1 h)); then W_o.  The last taps - 1 inputs of the convolutions are state as well.
+    Without ``decay_rank`` and ``gate_rank`` (both or neither): ONE decay a head from a product ``a`` [heads, width]
+    with ``dt_bias`` [heads], and the gate is a product ``g`` [heads * value_dim, width].  ``gate_act``: "sigmoid"
+    (default) or "silu".
     params: ``width``, ``n_heads``, ``n_qk_heads``, ``key_dim``, ``value_dim``, ``taps``, ``decay_rank``,
     ``gate_rank``, ``eps``.
     weights: ``q``, ``k`` [qk heads * key_dim, width], ``v`` [heads * value_dim, width], ``q_conv``, ``k_conv``,
@@ -118,34 +123,59 @@ class GatedDeltaRule(_StateMixer):
     UNIT_EPS = 1e-6  # inside the root of the unit norms of q and k; a constant of the mixer
 
     @classmethod
+    def _inputs(cls, params):
+        """The matrices that one product of the mixer's input serves, in the order of its columns."""
+        return ("q", "k", "v", "g", "b", "a") if cls._head_decay(params) else ("q", "k", "v", "b")
+
+    @staticmethod
+    def _head_decay(params) -> bool:
+        if (params.get("decay_rank") is None) != (params.get("gate_rank") is None):
+            raise ConfigError("a gated delta rule has low-rank products for both its decay and its gate, or for neither")
+        return params.get("decay_rank") is None
+
+    @classmethod
     def fused_weights(cls, params):
-        return {"qkvb": ("q", "k", "v", "b"), "a1g1": ("a1", "g1")}
+        if cls._head_decay(params):
+            return {"qkvgba": cls._inputs(params)}
+        return {"qkvb": cls._inputs(params), "a1g1": ("a1", "g1")}
 
     @classmethod
     def weight_shapes(cls, params):
-        d, nh, nq, kd, vd, taps, ra, rg = (params[k] for k in ("width", "n_heads", "n_qk_heads", "key_dim", "value_dim",
-                                                               "taps", "decay_rank", "gate_rank"))
-        return {"q": ((nq * kd, d), "matrix"), "k": ((nq * kd, d), "matrix"), "v": ((nh * vd, d), "matrix"),
-                "b": ((nh, d), "matrix"), "q_conv": ((nq * kd, taps), "vector"), "k_conv": ((nq * kd, taps), "vector"),
-                "v_conv": ((nh * vd, taps), "vector"), "A_log": ((nh,), "vector"), "a1": ((ra, d), "matrix"),
-                "a2": ((nh * kd, ra), "matrix"), "dt_bias": ((nh * kd,), "vector"), "g1": ((rg, d), "matrix"),
-                "g2": ((nh * vd, rg), "matrix"), "norm": ((vd,), "vector"), "o": ((d, nh * vd), "matrix")}
+        d, nh, nq, kd, vd, taps = (params[k] for k in ("width", "n_heads", "n_qk_heads", "key_dim", "value_dim", "taps"))
+        shapes = {"q": ((nq * kd, d), "matrix"), "k": ((nq * kd, d), "matrix"), "v": ((nh * vd, d), "matrix"),
+                  "b": ((nh, d), "matrix"), "q_conv": ((nq * kd, taps), "vector"), "k_conv": ((nq * kd, taps), "vector"),
+                  "v_conv": ((nh * vd, taps), "vector"), "A_log": ((nh,), "vector"), "norm": ((vd,), "vector"),
+                  "o": ((d, nh * vd), "matrix")}
+        if cls._head_decay(params):
+            shapes.update({"a": ((nh, d), "matrix"), "dt_bias": ((nh,), "vector"), "g": ((nh * vd, d), "matrix")})
+        else:
+            ra, rg = params["decay_rank"], params["gate_rank"]
+            shapes.update({"a1": ((ra, d), "matrix"), "a2": ((nh * kd, ra), "matrix"), "dt_bias": ((nh * kd,), "vector"),
+                           "g1": ((rg, d), "matrix"), "g2": ((nh * vd, rg), "matrix")})
+        return shapes
 
     def __init__(self, params, weights, dtype: DType, device):
-        self.n_heads, self.n_qk_heads, self.key_dim, self.value_dim, self.taps, self.decay_rank = (
-            int(params[k]) for k in ("n_heads", "n_qk_heads", "key_dim", "value_dim", "taps", "decay_rank"))
+        self.n_heads, self.n_qk_heads, self.key_dim, self.value_dim, self.taps = (
+            int(params[k]) for k in ("n_heads", "n_qk_heads", "key_dim", "value_dim", "taps"))
+        self.head_decay = self._head_decay(params)
+        self.decay_rank = int(params.get("decay_rank") or 0)
+        self.gate_act = params.get("gate_act", "sigmoid")
+        if self.gate_act not in ("sigmoid", "silu"):
+            raise ConfigError(f"a delta rule's gate {self.gate_act!r} is not sigmoid or silu")
         self.eps = float(params["eps"])
         if self.n_heads % self.n_qk_heads:
             raise ConfigError(f"{self.n_heads} heads are not a multiple of {self.n_qk_heads} q/k heads")
         if not (1 <= self.taps <= 9):
             raise ConfigError(f"a short convolution of {self.taps} taps is outside 1 to 9")
-        self.w_in = weights.get("qkvb")
+        self.w_in = weights.get("qkvgba" if self.head_decay else "qkvb")
         if self.w_in is None:
-            self.w_in = torch.cat([weights[r] for r in ("q", "k", "v", "b")], dim=0).contiguous()
-        self.w_low = weights.get("a1g1")
-        if self.w_low is None:
-            self.w_low = torch.cat([weights["a1"], weights["g1"]], dim=0).contiguous()
-        self.w_a2, self.w_g2, self.w_o = weights["a2"], weights["g2"], weights["o"]
+            self.w_in = torch.cat([weights[r] for r in self._inputs(params)], dim=0).contiguous()
+        self.w_o = weights["o"]
+        if not self.head_decay:
+            self.w_low = weights.get("a1g1")
+            if self.w_low is None:
+                self.w_low = torch.cat([weights["a1"], weights["g1"]], dim=0).contiguous()
+            self.w_a2, self.w_g2 = weights["a2"], weights["g2"]
         self.conv = torch.cat([_vector(weights[r]) for r in ("q_conv", "k_conv", "v_conv")], dim=0).contiguous()
         self.a_log, self.dt_bias, self.norm = _vector(weights["A_log"]), _vector(weights["dt_bias"]), _vector(weights["norm"])
         self.channels = 2 * self.n_qk_heads * self.key_dim + self.n_heads * self.value_dim
@@ -161,7 +191,9 @@ class GatedDeltaRule(_StateMixer):
         self._owning(owns_cache)
         nh, nq, kd, vd = self.n_heads, self.n_qk_heads, self.key_dim, self.value_dim
         n = h.shape[0]
-        p = linear(h, self.w_in, out_dtype=torch.float32)          # q | k | v | b
+        p = linear(h, self.w_in, out_dtype=torch.float32)          # q | k | v | b, or q | k | v | g | b | a
+        if self.head_decay:
+            return self._heads_out_one_decay(p, ctx, store)
         low = linear(h, self.w_low, out_dtype=self.act_dtype)      # a1 h | g1 h
         decay = linear(low[:, :self.decay_rank], self.w_a2, out_dtype=torch.float32)
         gate = linear(low[:, self.decay_rank:], self.w_g2, out_dtype=torch.float32)
@@ -174,7 +206,69 @@ class GatedDeltaRule(_StateMixer):
         ops.state_scan(o, qkv, qkv[:, nq * kd:], qkv[:, 2 * nq * kd:], decay, p[:, self.channels:], store[0].state,
                        ctx.cu_seqlens, ctx.seq_slot, nh, nq, kd, vd, delta=True, max_new=ctx.max_new)
         y = torch.empty((n, nh * vd), dtype=self.act_dtype, device=h.device)
-        ops.head_norm_gate(y, o, self.norm, gate, nh, vd, self.eps, "sigmoid")
+        ops.head_norm_gate(y, o, self.norm, gate, nh, vd, self.eps, self.gate_act)
+        return y
+
+    def _heads_out_one_decay(self, p, ctx, store):
+        nh, nq, kd, vd = self.n_heads, self.n_qk_heads, self.key_dim, self.value_dim
+        n = p.shape[0]
+        qkv = self._rows(ctx)((n, self.channels), dtype=torch.float32, device=p.device)
+        conv_state = store[1].state if self.taps > 1 else None
+        ops.short_conv(qkv, p, self.conv, conv_state, ctx.cu_seqlens, ctx.seq_slot, ctx.max_new, "silu")
+        o = self._rows(ctx)((n, nh * vd), dtype=torch.float32, device=p.device)
+        gate, beta = p[:, self.channels:], p[:, self.channels + nh * vd:]
+        ops.head_scan(o, qkv, qkv[:, nq * kd:], qkv[:, 2 * nq * kd:], store[0].state, ctx.cu_seqlens, ctx.seq_slot, nh, nq,
+                      kd, vd, decay_raw=beta[:, nh:], a_log=self.a_log, dt_bias=self.dt_bias, beta=beta,
+                      q_scale=kd ** -0.5, unit_eps=self.UNIT_EPS, max_new=ctx.max_new)
+        y = torch.empty((n, nh * vd), dtype=self.act_dtype, device=p.device)
+        ops.head_norm_gate(y, o, self.norm, gate, nh, vd, self.eps, self.gate_act)
+        return y
+
+
+class ConstantDecayLinearAttention(_StateMixer):
+    """q = silu(W_q h), k = silu(W_k h), v = silu(W_v h), head by head; S_t = decay_h S_(t-1) + k_t v_t^T,
+    o_t = S_t^T q_t with one constant decay a head and no other scale; the heads side by side are RMS-normed together,
+    times the weight ``norm``, times sigmoid(W_g h); then W_o.
+    params: ``width``, ``n_heads``, ``key_dim``, ``value_dim``, ``decay`` (a number a head), ``eps``.
+    weights: ``q``, ``k`` [heads * key_dim, width], ``v``, ``g`` [heads * value_dim, width], ``norm``
+    [heads * value_dim], ``o`` [width, heads * value_dim]."""
+
+    @classmethod
+    def fused_weights(cls, params):
+        return {"qkvg": ("q", "k", "v", "g")}
+
+    @classmethod
+    def weight_shapes(cls, params):
+        d, nh, kd, vd = (params[k] for k in ("width", "n_heads", "key_dim", "value_dim"))
+        return {"q": ((nh * kd, d), "matrix"), "k": ((nh * kd, d), "matrix"), "v": ((nh * vd, d), "matrix"),
+                "g": ((nh * vd, d), "matrix"), "norm": ((nh * vd,), "vector"), "o": ((d, nh * vd), "matrix")}
+
+    def __init__(self, params, weights, dtype: DType, device):
+        self.n_heads, self.key_dim, self.value_dim = (int(params[k]) for k in ("n_heads", "key_dim", "value_dim"))
+        self.eps = float(params["eps"])
+        decay = [float(d) for d in params["decay"]]
+        if len(decay) != self.n_heads:
+            raise ConfigError(f"{len(decay)} decays for {self.n_heads} heads")
+        self.decay = torch.tensor(decay, dtype=torch.float32, device=device)
+        self.w_in = weights.get("qkvg")
+        if self.w_in is None:
+            self.w_in = torch.cat([weights[r] for r in ("q", "k", "v", "g")], dim=0).contiguous()
+        self.w_o, self.norm = weights["o"], _vector(weights["norm"])
+        self.act_dtype = torch_dtype(dtype)
+
+    def cache_need(self):
+        return StateNeed((self.n_heads, self.value_dim, self.key_dim), "float32")
+
+    def heads_out(self, h, ctx, store, owns_cache=True):
+        self._owning(owns_cache)
+        nh, kd, vd = self.n_heads, self.key_dim, self.value_dim
+        n = h.shape[0]
+        p = linear(h, self.w_in, out_dtype=torch.float32)   # q | k | v | g
+        o = self._rows(ctx)((n, nh * vd), dtype=torch.float32, device=h.device)
+        ops.head_scan(o, p, p[:, nh * kd:], p[:, 2 * nh * kd:], store.state, ctx.cu_seqlens, ctx.seq_slot, nh, nh, kd, vd,
+                      decay=self.decay, silu=True, max_new=ctx.max_new)
+        y = torch.empty((n, nh * vd), dtype=self.act_dtype, device=h.device)
+        ops.head_norm_gate(y, o, self.norm, p[:, 2 * nh * kd + nh * vd:], 1, nh * vd, self.eps, "sigmoid")
         return y
 
 
@@ -238,3 +332,4 @@ class DecayRemovalRule(_StateMixer):
 register_part("mixer", "decay_removal_rule", DecayRemovalRule)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
+register_part("mixer", "constant_decay_linear_attention", ConstantDecayLinearAttention)

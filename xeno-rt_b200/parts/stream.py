@@ -74,6 +74,25 @@ class AddRow:
         return x
 
 
+class AddEmbedding:
+    """x <- x + x0 in 32-bit, in place: what the embedding gave is added to the stream once more (at the beginning of a
+    further pass over a stretch of layers).  params: ``width``.  No weights."""
+
+    graph_safe = True
+
+    @classmethod
+    def weight_shapes(cls, params):
+        return {}
+
+    def __init__(self, params, weights, dtype, device):
+        self.width = int(params["width"])
+
+    def forward(self, x, x0, ctx):
+        ops.stream_add(x, x0)
+        return x
+
+
+register_part("stream", "add_embedding", AddEmbedding)
 register_part("stream", "add_row", AddRow)
 register_part("stream", "mix_with_embedding", MixWithEmbedding)
 register_part("stream", "rmsnorm", NormedStream)

@@ -1,0 +1,418 @@
+"""The Zivovik decoder through the library's engine, cache and entry points, against the plain implementation
+(tests/plain/zivovik.py): the residual stream after every layer run, whole prompts, token-by-token decoding, prompts cut
+into portions down to two tokens, batches of unequal requests, slots and blocks that are used again, long decoding
+through captured steps, the last position of the table, configurations drawn at random, greedy generation through the
+scheduler, the command line and the trace replay program."""
+import copy
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+
+from helpers import random_prompts, scaled_error
+from plain import zivovik as plain
+from plain.files import read_model_folder
+from zivovik_cases import CASES, make_case, random_config, random_weights, write_folder
+
+pytestmark = pytest.mark.gpu
+# Of the logit scale.  The 32-bit runs are the sharp ones: a wrong key, a temperature's step that is one token off, a lost
+# state or a missing row of the position table moves the logits by far more (a test below says by how much).  In bfloat16
+# a close call between two experts may go the other way than in the plain model, so single positions may move further
+# than the rest: the worst position, nearly all positions and the median have bounds of their own.
+TOL = {"float32": 4e-5, "bfloat16": 0.2}
+MOST = {"float32": 4e-5, "bfloat16": 0.05}      # 96 of 100 positions
+MEDIAN = {"float32": 1e-5, "bfloat16": 0.02}
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+
+
+@pytest.fixture(scope="module")
+def cases(tmp_path_factory):
+    root = tmp_path_factory.mktemp("zivovik")
+    return {name: make_case(root, name) for name in CASES}
+
+
+def _check(got, want, dtype, rows=None):
+    rows = list(range(len(got))) if rows is None else list(rows)
+    err = np.abs(got.astype(np.float64) - want[rows]).max(-1) / np.abs(want).max()
+    assert np.isfinite(err).all() and err.max() < TOL[dtype], (err.max(), rows[int(np.argmax(err))])
+    if len(err) >= 20:
+        assert np.quantile(err, 0.96) < MOST[dtype] and np.median(err) < MEDIAN[dtype], (np.quantile(err, 0.96), np.median(err))
+
+
+def _engine(folder, dtype, tokens=64 * 24):
+    from xeno_rt_b200.engine import Engine
+    from xeno_rt_b200.engine.model import Model
+    return Engine(Model.load(folder, dtype=dtype), tokens)
+
+
+def _run_cut(engine, tokens, cuts):
+    from xeno_rt_b200.engine import StepEntry
+    slot = engine.open_slot()
+    parts, at = [], 0
+    for size in cuts:
+        parts.append(engine.step([StepEntry(slot, tokens[at:at + size], list(range(size)))]).cpu().numpy())
+        at += size
+    assert at == len(tokens)
+    engine.close_slot(slot)
+    return np.concatenate(parts)
+
+
+@pytest.mark.parametrize("name", list(CASES))
+def test_the_stream_after_every_layer_run_is_the_plain_one(cases, name):
+    """In 32-bit, layer run by layer run: the first that differs names the mechanism at fault."""
+    import torch
+    from xeno_rt_b200.engine import StepEntry
+    folder, config, weights = cases[name]
+    engine = _engine(folder, "float32")
+    model = engine.model
+    kept, original = [], list(model.arrangements)
+
+    def wrap(fn):
+        def run(parts, x, ctx, stores, owns):
+            fn(parts, x, ctx, stores, owns)
+            kept.append(x.clone())
+        run.first_norm = fn.first_norm
+        return run
+    model.arrangements = [wrap(fn) for fn in original]
+    tokens = random_prompts(config["vocab"], [150], seed=2)[0]
+    want = []
+    plain.forward(config, weights, tokens, layers_out=want)
+    slot = engine.open_slot()
+    engine.step([StepEntry(slot, tokens, [0])])
+    engine.close_slot(slot)
+    model.arrangements = original
+    assert len(kept) == len(want) == len(plain.order(config))
+    for i, (got, ref) in enumerate(zip(kept, want)):
+        assert got.dtype == torch.float32  # the stream itself is 32-bit
+        assert np.abs(got.cpu().numpy() - ref).max() < 4e-5 * max(1.0, np.abs(ref).max()), i
+
+
+def _mixers(config):
+    for layer in config["layers"]:
+        yield layer["type"], layer["mixer"]
+
+
+def _faults(config, weights):
+    """(name, config, weights) of models with one mechanism slightly off."""
+    steps = copy.deepcopy(config)
+    for kind, m in _mixers(steps):
+        for a in (m, m.get("left") or {}):
+            if a.get("q_temp"):
+                a["q_temp"]["every"] += 1
+    yield "the temperature steps one token later", steps, weights
+    decays = copy.deepcopy(config)
+    for kind, m in _mixers(decays):
+        if kind == "lightning":
+            m["decay"] = [0.999 * d for d in m["decay"]]
+    yield "decays 0.1 % smaller", decays, weights
+    loop = copy.deepcopy(config)
+    loop["loop"]["times"] += 1
+    yield "one pass more", loop, weights
+    yield "norm weights as they are stored", config, {k: (v - 1 if ".norm1" in k or ".norm2" in k else v) for k, v in weights.items()}
+    yield "positions one further", config, {k: (np.roll(v, -1, axis=0) if k == "pos" else v) for k, v in weights.items()}
+    yield "no write factor", config, {k: (0 * v if k.endswith("right.b") else v) for k, v in weights.items()}
+    yield "the convolution's oldest tap left out", config, {
+        k: (np.concatenate([0 * v[:, :1], v[:, 1:]], axis=1) if k.endswith(".conv") else v) for k, v in weights.items()}
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", list(CASES))
+def test_prompts_portions_and_decoding_give_the_plain_logits(cases, name, dtype):
+    folder, config, weights = cases[name]
+    engine = _engine(folder, dtype)
+    n = 330 if name == "wide" else 230
+    tokens = random_prompts(config["vocab"], [n], seed=1)[0]
+    want = plain.forward(config, weights, tokens)
+    if dtype == "float32" and name == "mixed":  # what a fault would look like here
+        for fault, other, others in _faults(config, weights):
+            off = plain.forward(other, others, tokens)
+            assert np.abs(off - want).max() / np.abs(want).max() > 20 * TOL[dtype], fault
+    whole = _run_cut(engine, tokens, [n])
+    _check(whole, want, dtype)
+    # most of it in one step, the rest token by token, across a block's edge
+    decoded = _run_cut(engine, tokens, [n - 100] + [1] * 100)
+    _check(decoded, want, dtype)
+    # portions of several sizes, down to two tokens and one
+    cuts = [2, 1, 2, 3, 59, 64, 5, 2]
+    portions = _run_cut(engine, tokens, cuts + [n - sum(cuts)])
+    _check(portions, want, dtype)
+    # token by token from the first one
+    _check(_run_cut(engine, tokens[:70], [1] * 70), want[:70], dtype)
+    if dtype == "float32":  # how the tokens are cut changes nothing but rounding
+        assert scaled_error(decoded, whole) < 1e-5 and scaled_error(portions, whole) < 1e-5
+    engine.check_errors()
+    engine.cache.check()
+    assert engine.cache.blocks_free() == engine.cache.n_blocks
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["mixed", "odd"])
+def test_unequal_batches_equal_each_request_alone_and_slots_are_used_again(cases, name, dtype):
+    from xeno_rt_b200.engine import StepEntry
+    folder, config, weights = cases[name]
+    engine = _engine(folder, dtype, 64 * 16)
+    lengths = [1, 150, 7, 66, 129]
+    decode = 12
+    prompts = random_prompts(config["vocab"], [k + decode for k in lengths], seed=4)
+    want = [plain.forward(config, weights, p) for p in prompts]
+    alone = _run_cut(engine, prompts[3], [lengths[3]] + [1] * decode)
+    for turn in range(2):  # the second turn takes the slots and blocks that the first gave back, in another order
+        slots = [engine.open_slot() for _ in prompts]
+        if turn:
+            slots = slots[::-1]
+        got = [[] for _ in prompts]
+        out = engine.step([StepEntry(s, p[:k], list(range(k))) for s, p, k in zip(slots, prompts, lengths)]).cpu().numpy()
+        at = 0
+        for i, k in enumerate(lengths):
+            got[i].append(out[at:at + k])
+            at += k
+        live = list(range(len(prompts)))
+        for step in range(decode):
+            if step == 5:  # a shorter request ends earlier; its slot is closed while the others go on
+                engine.close_slot(slots[live.pop(0)])
+            out = engine.step([StepEntry(slots[i], [prompts[i][lengths[i] + step]], [0]) for i in live]).cpu().numpy()
+            for row, i in enumerate(live):
+                got[i].append(out[row:row + 1])
+        for i in live:
+            engine.close_slot(slots[i])
+        for i in range(len(prompts)):
+            _check(np.concatenate(got[i]), want[i], dtype)
+        if dtype == "float32":  # what else is in the batch changes nothing but rounding
+            assert scaled_error(np.concatenate(got[3]), alone) < 1e-5
+        engine.cache.check()
+        assert engine.cache.blocks_free() == engine.cache.n_blocks
+    engine.check_errors()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_step_may_mix_portions_and_single_tokens(cases, dtype):
+    """Requests that begin, go on by several tokens and go on by one, in one step: every state ends where its request's
+    portion ends."""
+    from xeno_rt_b200.engine import StepEntry
+    folder, config, weights = cases["mixed"]
+    engine = _engine(folder, dtype)
+    prompts = random_prompts(config["vocab"], [90, 77, 40], seed=14)
+    plans = [[30, 1, 1, 58], [1, 1, 70, 5], [3, 34, 1, 2]]
+    want = [plain.forward(config, weights, p) for p in prompts]
+    slots = [engine.open_slot() for _ in prompts]
+    at, got = [0, 0, 0], [[], [], []]
+    for step in range(4):
+        sizes = [plan[step] for plan in plans]
+        out = engine.step([StepEntry(s, p[a:a + k], list(range(k))) for s, p, a, k in zip(slots, prompts, at, sizes)]).cpu().numpy()
+        row = 0
+        for i, k in enumerate(sizes):
+            got[i].append(out[row:row + k])
+            row += k
+            at[i] += k
+    for g, w in zip(got, want):
+        _check(np.concatenate(g), w, dtype)
+    engine.check_errors()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_long_decoding_through_captured_steps_to_the_tables_last_position(cases, dtype):
+    """415 single-token steps after a short prompt, up to the last row of the position table; a step beyond it is refused
+    before anything runs, and the sequence stays usable."""
+    from xeno_rt_b200.core import XrtError
+    from xeno_rt_b200.engine import StepEntry
+    folder, config, weights = cases["mixed"]
+    engine = _engine(folder, dtype)
+    assert engine.use_graphs and engine.model.graph_safe
+    most = config["max_positions"]
+    tokens = random_prompts(config["vocab"], [most], seed=9)[0]
+    want = plain.forward(config, weights, tokens)
+    slot = engine.open_slot()
+    rows = [engine.step([StepEntry(slot, tokens[:5], list(range(5)))]).cpu().numpy()]
+    rows += [engine.step([StepEntry(slot, [t], [0])]).cpu().numpy() for t in tokens[5:]]
+    _check(np.concatenate(rows), want, dtype)
+    with pytest.raises(XrtError):
+        engine.step([StepEntry(slot, [1], [0])])
+    engine.close_slot(slot)
+    engine.cache.check()
+    assert engine.cache.blocks_free() == engine.cache.n_blocks
+    engine.check_errors()
+
+
+def test_what_the_cache_holds(cases):
+    """Keys and values for an attention, a matrix a head for a lightning layer, all of it and the convolution's inputs for
+    a parallel one; every pass of the loop its own."""
+    from xeno_rt_b200.engine.model import Model
+    folder, config, weights = cases["mixed"]
+    needs = [n["mixer"] for n in Model.load(folder, dtype="bfloat16").cache_needs()]
+    assert len(needs) == 7
+    assert tuple(needs[0].shape) == (3, 24, 16) and tuple(needs[6].shape) == (2, 8, 32)
+    assert [(n.n_kv_heads, n.head_dim, n.window) for n in (needs[1], needs[3], needs[5])] == [(2, 16, None), (2, 16, None), (1, 48, None)]
+    for n in (needs[2], needs[4]):
+        keys, (state, conv) = n
+        assert (keys.n_kv_heads, keys.head_dim) == (2, 32)
+        assert tuple(state.shape) == (4, 32, 16) and tuple(conv.shape) == (3, 2 * 2 * 16 + 4 * 32) and state.dtype == "float32"
+    folder, config, weights = cases["odd"]
+    needs = [n["mixer"] for n in Model.load(folder, dtype="float32").cache_needs()]
+    assert len(needs[0][1]) == 1 and tuple(needs[0][1][0].shape) == (3, 20, 12)   # one tap: nothing before the token is needed
+
+
+@pytest.mark.parametrize("seed", range(10))
+def test_configurations_drawn_at_random(tmp_path, seed):
+    from xeno_rt_b200.engine import StepEntry
+    rng = np.random.default_rng(2000 + seed)
+    config = random_config(rng)
+    weights = random_weights(config, seed)
+    folder = write_folder(str(tmp_path / "m"), config, weights)
+    n = 170
+    tokens = random_prompts(config["vocab"], [n], seed=seed)[0]
+    want = plain.forward(config, weights, tokens)
+    for dtype in ("float32", "bfloat16"):
+        engine = _engine(folder, dtype)
+        for cuts in ([n], [n - 60] + [1] * 60, [2, 1, 63, 2, 66, n - 134]):
+            _check(_run_cut(engine, tokens, cuts), want, dtype)
+        # three unequal requests together: prompts of the same tokens, cut at different places, then decoded
+        starts = [3, 64, 130]
+        slots = [engine.open_slot() for _ in starts]
+        out = engine.step([StepEntry(s, tokens[:k], [k - 1]) for s, k in zip(slots, starts)]).cpu().numpy()
+        _check(out, want, dtype, [k - 1 for k in starts])
+        for j in range(5):
+            out = engine.step([StepEntry(s, [tokens[k + j]], [0]) for s, k in zip(slots, starts)]).cpu().numpy()
+            _check(out, want, dtype, [k + j for k in starts])
+        engine.check_errors()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_greedy_generation_through_the_scheduler(cases, dtype):
+    from xeno_rt_b200 import GenerateRequest, Runtime
+    folder, config, weights = cases["mixed"]
+    prompts = random_prompts(config["vocab"], [3, 70, 20], seed=6)
+    session = Runtime.load(folder, dtype=dtype).new_session()
+    requests = [GenerateRequest(p, max_tokens=10, temperature=0.0, repetition_penalty=1.0, stop_ids=()) for p in prompts]
+    results, stats = session.generate_batch(requests)
+    tol = MOST[dtype]
+    for p, r in zip(prompts, results):
+        assert len(r.tokens) == 10 and r.finish_reason == "length"
+        want = plain.forward(config, weights, list(p) + list(r.tokens))
+        scale = np.abs(want).max()
+        for i, token in enumerate(r.tokens):  # the plain model's best token wherever its lead is beyond rounding
+            row = want[len(p) + i - 1]
+            top = np.sort(row)[-2:]
+            if top[1] - top[0] > 2 * tol * scale:
+                assert int(token) == int(np.argmax(row)), (i, token)
+    session.backend.engine.cache.check()
+
+
+def test_the_command_line_generates_what_the_session_generates(cases):
+    """``xrt generate --model DIR`` picks the design by config.json: greedy tokens equal the session's."""
+    from xeno_rt_b200 import GenerateRequest, Runtime
+    folder, config, _ = cases["odd"]
+    prompts = random_prompts(config["vocab"], [4, 31], seed=8)
+    xrt = [sys.executable, os.path.join(ROOT, "bin", "xrt"), "generate", "--model", folder, "--dtype", "float32",
+           "--max-tokens", "9", "--stop-ids", "", "--prompt-ids", ",".join(map(str, prompts[0])),
+           "--prompt-ids", ",".join(map(str, prompts[1])), "--temperature", "0", "--repetition-penalty", "1.0"]
+    greedy = subprocess.run(xrt, capture_output=True, text=True, timeout=600)
+    assert greedy.returncode == 0, greedy.stderr
+    session = Runtime.load(folder, dtype="float32").new_session()
+    results, _ = session.generate_batch([GenerateRequest(p, max_tokens=9, temperature=0.0, repetition_penalty=1.0,
+                                                         stop_ids=()) for p in prompts])
+    lines = [list(map(int, l.split(","))) for l in greedy.stdout.strip().splitlines() if l]
+    assert lines == [list(r.tokens) for r in results]
+
+
+def test_a_model_without_a_file_is_drawn_from_a_seed():
+    from xeno_rt_b200.engine import Engine, StepEntry
+    from xeno_rt_b200.engine.model import Model
+    engine = Engine(Model.random(CASES["odd"][0], seed=1), 256)
+    slot = engine.open_slot()
+    a = engine.step([StepEntry(slot, [1, 2, 3, 4], [3])])
+    b = engine.step([StepEntry(slot, [5], [0])])
+    assert a.shape == (1, CASES["odd"][0]["vocab"]) and bool(a.isfinite().all()) and bool(b.isfinite().all())
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_trace_replay_as_a_user_runs_it(cases, tmp_path, dtype):
+    """``bin/trace_run`` on a Zivovik folder: five requests of unequal lengths start as one batch and are decoded
+    together, the shorter ones end earlier."""
+    folder, config, weights = cases["odd"]
+    lengths, tails = [3, 70, 1, 65, 20], [4, 9, 2, 9, 6]
+    prompts = random_prompts(config["vocab"], [k + t for k, t in zip(lengths, tails)], seed=21)
+    want = [plain.forward(config, weights, p) for p in prompts]
+    steps = [{"step": 0, "entries": [{"id": f"q{i}", "tokens": p[:k], "want": list(range(k))}
+                                     for i, (p, k) in enumerate(zip(prompts, lengths))], "end": []}]
+    for n in range(max(tails)):
+        live = [i for i, t in enumerate(tails) if n < t]
+        steps.append({"step": n + 1, "entries": [{"id": f"q{i}", "tokens": [prompts[i][lengths[i] + n]],
+                                                  "want": [0] if n % 2 == 0 else []} for i in live],
+                      "end": [f"q{i}" for i in live if n == tails[i] - 1]})
+    out = tmp_path / dtype
+    proc = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", folder, "--dtype", dtype, "--out", str(out),
+                           "--max-tokens", str(sum(len(p) for p in prompts))],
+                          input="\n".join(json.dumps(s) for s in steps) + "\n", capture_output=True, text=True, timeout=900)
+    assert proc.returncode == 0, proc.stderr
+    assert [l for l in proc.stdout.splitlines() if l.startswith("done")] == [f"done {s['step']}" for s in steps]
+    got, rows = {i: [] for i in range(len(prompts))}, {i: [] for i in range(len(prompts))}
+    for s in steps:
+        wanted = sum(len(e["want"]) for e in s["entries"])
+        if not wanted:
+            assert not (out / f"{s['step']}.f32").exists()
+            continue
+        data = np.fromfile(out / f"{s['step']}.f32", dtype="<f4").reshape(-1, config["vocab"])
+        assert data.shape[0] == wanted
+        at = 0
+        for e in s["entries"]:
+            i = int(e["id"][1:])
+            first = 0 if s["step"] == 0 else lengths[i] + s["step"] - 1
+            got[i].append(data[at:at + len(e["want"])])
+            rows[i] += [first + w for w in e["want"]]
+            at += len(e["want"])
+    for i in range(len(prompts)):
+        _check(np.concatenate(got[i]), want[i], dtype, rows[i])
+
+
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+def test_a_captured_step_of_many_sequences_leaves_the_padding_rows_states_alone(cases, name):
+    """Eleven sequences a step (16 rows with padding), then 19: every sequence's state goes its own way."""
+    from xeno_rt_b200.engine import StepEntry
+    folder, config, weights = cases[name]
+    engine = _engine(folder, "bfloat16", 64 * 24)
+    lengths = [3, 9, 17, 5, 11, 2, 8, 13, 4, 6, 21, 1, 7, 12, 30, 10, 2, 3, 5]
+    decode = 5
+    prompts = random_prompts(config["vocab"], [k + decode for k in lengths], seed=12)
+    want = [plain.forward(config, weights, p) for p in prompts]
+    for count in (11, 19):
+        slots = [engine.open_slot() for _ in range(count)]
+        out = engine.step([StepEntry(s, p[:k], [k - 1]) for s, p, k in zip(slots, prompts, lengths)]).cpu().numpy()
+        for i in range(count):
+            _check(out[i:i + 1], want[i], "bfloat16", [lengths[i] - 1])
+        for step in range(decode):
+            out = engine.step([StepEntry(slots[i], [prompts[i][lengths[i] + step]], [0]) for i in range(count)]).cpu().numpy()
+            for i in range(count):
+                _check(out[i:i + 1], want[i], "bfloat16", [lengths[i] + step])
+        for s in slots:
+            engine.close_slot(s)
+    engine.check_errors()
+    engine.cache.check()
+
+
+def test_one_far_key_among_hundreds_decides_the_logits(tmp_path):
+    """A model of one attention layer in which the last token's query is the first token's key many times over (that score
+    stands out by far): the output follows the first token's value through a prompt, portions and decoding, and another
+    first token changes the last logits."""
+    from zivovik_cases import attn, layer, model, temp
+    config = model(40, 32, [layer("attention", attn(2, 1, 16, 1.5, temp(0.5, 64)), None)], scale=0.5, mult=2.0)
+    weights = random_weights(config, 5)
+    weights["pos"] = 0 * weights["pos"]
+    h = plain.offset_norm(0.5 * weights["embed"].astype(np.float64), weights["l0.norm1"], 1e-5)
+    key = weights["l0.mix.k"].astype(np.float64) @ h[7]
+    match = np.outer(key, h[5]) / (h[5] @ h[5])
+    weights["l0.mix.q"] = np.concatenate([match, match]).astype(np.float32)
+    folder = write_folder(str(tmp_path / "m"), config, weights)
+    rng = np.random.default_rng(3)
+    tokens = [7] + [int(t) for t in rng.integers(8, 40, 300)] + [5]
+    w = read_model_folder(folder)[1]    # as the file rounds them
+    want = plain.forward(config, w, tokens)
+    without = plain.forward(config, w, [9] + tokens[1:])
+    assert np.abs(want[-1] - without[-1]).max() > 0.2 * np.abs(want).max()
+    for dtype in ("float32", "bfloat16"):
+        engine = _engine(folder, dtype)
+        for cuts in ([302], [301, 1], [64, 2, 1, 61, 64, 110], [250] + [1] * 52):
+            got = _run_cut(engine, tokens, cuts)
+            assert np.abs(got[-1] - want[-1]).max() < (1e-4 if dtype == "float32" else 0.02) * np.abs(want).max(), (dtype, cuts)

@@ -98,6 +98,8 @@ class GroupedQueryAttention:
         hd, vd, size = cls._sizes(params)
         if hd != size or vd != size or not params.get("own_kv", True):
             return {}  # the part lays the heads out itself
+        if params.get("gate") == "sigmoid_head" and int(params["n_heads"]) % 4:
+            return {}  # the part rounds the product's row up to whole 16 bytes
         if params.get("tied_values"):
             return {"qkg": ("q", "k", "g")} if params.get("gate") else {"qk": ("q", "k")}
         return {"qkvg": ("q", "k", "v", "g")} if params.get("gate") else {"qkv": ("q", "k", "v")}
@@ -191,6 +193,9 @@ class GroupedQueryAttention:
                     pieces.append(_pad_rows(weights["v"], self.n_kv_heads, true_vdim, self.head_dim))
             if self.gate == "sigmoid_head":
                 pieces.append(weights["g"])
+                odd = -self.n_heads % 4  # rows of whole 16 bytes, which the kernels that read the product's row ask for
+                if odd:
+                    pieces.append(torch.zeros((odd, self.width), dtype=weights["g"].dtype, device=weights["g"].device))
             elif self.gate:
                 pieces.append(_pad_rows(weights["g"], self.n_heads, true_vdim, self.head_dim))
             self.w_qkv = torch.cat(pieces, dim=0).contiguous()

@@ -79,7 +79,7 @@ def decode_from_qkv(out, qkv, k_offset, v_offset, q_norm, k_norm, eps, cos_sin, 
     the rotation and the cache write itself (one kernel and one boundary less a layer).  False where that
     kernel does not take the case; the caller then runs the rotation kernel and ``run``."""
     rope_half = 0 if cos_sin is None else cos_sin.shape[1]
-    if not (ctx.all_single and ctx.n_tokens <= 65535
+    if not (ctx.all_single and ctx.n_tokens <= 65535 and qkv.shape[1] % 4 == 0  # rows of whole 16 bytes
             and ops.attention_decode_takes_qkv(n_heads, n_kv_heads, head_dim, rope_half, pairing)):
         return False
     chunk, n_splits, clusters = _decode_split_of(ctx, n_kv_heads, qkv.device, window or mask_chunk)

@@ -398,10 +398,27 @@ def fadutar_config(width: int, heads: int, kv_heads: int, head_dim: int, inner: 
     return {"architecture": "Fadutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": out}
 
 
+def zivovik_config(width: int, heads: int, kv_heads: int, head_dim: int, inner: int, layers: int, vocab: int) -> dict:
+    """A Zivovik model at the sizes of a dense decoder of that width: layers go parallel, attention, lightning, attention,
+    and again; every layer with 16 experts of ``inner`` / 8 units of which a token uses 2.  Attention (also the left
+    half of a parallel mixer) has ``heads`` x ``head_dim`` with ``kv_heads`` kv heads; the delta rule (its right half)
+    ``heads`` heads with keys and values of ``head_dim``, half as many q/k heads and 4 taps; lightning attention ``heads``
+    heads of ``head_dim``; the first two layers are a loop that runs once."""
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+            "q_temp": {"coef": 0.1, "every": 1024}}
+    right = {"heads": heads, "kv_heads": max(1, heads // 2), "dim": head_dim, "vdim": head_dim, "conv": 4}
+    lightning = {"heads": heads, "dim": head_dim, "vdim": head_dim, "decay": [1.0 - 2.0 ** (-2 - 8.0 * h / heads) for h in range(heads)]}
+    moe = {"kind": "moe", "expert": {"ff": inner // 8}, "router": {"experts": 16, "top": 2}}
+    pattern = [("parallel", {"left": attn, "right": right}), ("attention", attn), ("lightning", lightning), ("attention", attn)]
+    return {"architecture": "Zivovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0},
+            "residual_mult": 0.5, "max_positions": 1 << 14, "loop": {"start": 0, "stop": min(2, layers), "times": 1},
+            "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in (pattern[i % 4] for i in range(layers))]}
+
+
 DESIGN_CONFIGS = {"givopel": givopel_config, "guzuvik": guzuvik_config, "zogevik": zogevik_config,
-                  "sofunex": sofunex_config, "fadutar": fadutar_config}
+                  "sofunex": sofunex_config, "fadutar": fadutar_config, "zivovik": zivovik_config}
 # the library's model that is closest to a design, timed beside it at equal sizes (besides the dense decoder)
-DESIGN_NEIGHBOUR = {"zogevik": "guzuvik", "sofunex": "givopel", "fadutar": "zogevik"}
+DESIGN_NEIGHBOUR = {"zogevik": "guzuvik", "sofunex": "givopel", "fadutar": "zogevik", "zivovik": "givopel"}
 
 DESIGN_SIZES = {
     # name: (width, heads, kv heads, head size, feed-forward width, vocabulary)

@@ -23,7 +23,7 @@ __global__ void swiglu_kernel(TO* __restrict__ out, const TI* __restrict__ gate_
 template <typename TO>
 __global__ void relu_squared_kernel(TO* __restrict__ out, const float* __restrict__ x, size_t total) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x);
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const float v = fmaxf(x[i], 0.f);
     out[i] = from_float<TO>(v * v);

@@ -148,7 +148,7 @@ attention_decode_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
   constexpr int D_TILES = HD_MAX / 8;
   extern __shared__ __align__(16) unsigned char smem[];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(q, k_pool, v_pool, tok_slot, tok_pos, block_table, sinks);
   const int split = blockIdx.x, kv_head = blockIdx.y, tok = blockIdx.z;
   const int slot = tok_slot[tok];
   if (slot < 0) {  // a padding row: zeros (with several splits and no counters the combine kernel writes them)
@@ -296,7 +296,7 @@ __global__ void attention_combine_kernel(__nv_bfloat16* __restrict__ out, const 
                                          const KeyRange range, int chunk, int n_splits,
                                          const float* __restrict__ sinks) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(part_o, part_ml, tok_slot, tok_pos, sinks);
   const int lane = threadIdx.x & 31, pieces = (head_dim + COMBINE_DIMS - 1) / COMBINE_DIMS;
   const int warp_global = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int row = warp_global / pieces;  // (token, head)
@@ -425,7 +425,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   const int group = n_heads / n_kv_heads;
   if (slot < 0) {  // a padding row: zeros (with several splits and no counters the combine kernel writes them)
     // (the same for every block of a cluster: all of them leave here, none waits for another)
-    pdl_wait();
+    pdl_wait(q, tok_slot, tok_pos, block_table, sinks);
     if (n_splits == 1 || ((counters != nullptr || clustered) && split == 0)) {
       __nv_bfloat16* dst = out + ((size_t)tok * n_heads + (size_t)kv_head * group) * head_dim;
       for (int i = threadIdx.x; i < group * head_dim; i += blockDim.x) dst[i] = __float2bfloat16_rn(0.f);
@@ -437,7 +437,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   const int begin = split_begin(split, chunk, first_key);
   const int end = split_end(split, chunk, first_key, len);
   const bool has_keys = begin < end;
-  if (!has_keys && !clustered) { pdl_wait(); return; }  // this split holds no visible key: the combine step skips it too
+  if (!has_keys && !clustered) { pdl_wait(q, tok_slot, tok_pos, block_table, sinks); return; }  // this split holds no visible key: the combine step skips it too
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int boxes = head_dim / 64;
@@ -492,7 +492,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
   // (A layer that reads another layer's cache has a newest key that a kernel of this step wrote.)
   const bool early = has_keys && ((fused.qkv != nullptr && fused.k_pool != nullptr) || begin + XRT_BLOCK_TOKENS <= len - 1);
   if (asks && early) issue_tile(0, 0, block_of(0));
-  pdl_wait();
+  pdl_wait(q, tok_slot, tok_pos, block_table, sinks);
   uint32_t qb[D_TILES / 2][2];
   if (fused.qkv == nullptr) {
     const __nv_bfloat16* qt = q + ((size_t)tok * n_heads + (size_t)kv_head * group) * head_dim;

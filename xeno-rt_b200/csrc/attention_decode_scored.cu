@@ -180,7 +180,7 @@ __global__ void attention_decode_scored_merge_kernel(__nv_bfloat16* __restrict__
                                                      const int* __restrict__ tok_slot, int n_heads, int head_dim,
                                                      int n_splits, const ScoreOptions opt) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(partial, tok_slot);
   const int t = blockIdx.x, head = blockIdx.y;
   if (tok_slot[t] < 0) return;  // the first kernel wrote the padding row's zeros
   const float* from = partial + ((size_t)t * n_heads + head) * n_splits * (head_dim + 2);

@@ -251,6 +251,18 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
 __device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 
+// The wait, for a kernel with `const T* __restrict__` parameters: such a parameter tells the compiler that what it points
+// to never changes while the kernel runs, so that it may move a load through it ahead of the wait, to where the kernel
+// before has not written yet.  The pointers are named here and come out of the wait as values of unknown origin: loads
+// written after the wait stay after it.  (Loads written before it, of what no kernel of the step writes, stay before.)
+template <typename P>
+__device__ __forceinline__ void forget_origin(P& pointer) { asm volatile("" : "+l"(pointer)::"memory"); }
+template <typename... P>
+__device__ __forceinline__ void pdl_wait(P&... pointers) {
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  (forget_origin(pointers), ...);
+}
+
 inline bool pdl_enabled() { return tuning().pdl; }
 
 template <typename... KArgs, typename... Args>

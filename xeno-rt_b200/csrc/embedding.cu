@@ -13,7 +13,7 @@ __global__ void embedding_kernel(float* __restrict__ out, const TW* __restrict__
                                  int* __restrict__ error_flag, float scale, const TW* __restrict__ pos_table,
                                  const int* __restrict__ positions, int n_positions) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(table, ids, pos_table, positions);
   const int t = blockIdx.x;
   const int id = ids[t];
   const int at = pos_table != nullptr ? positions[t] : 0;
@@ -34,7 +34,7 @@ __global__ void embedding_vec_kernel(float* __restrict__ out, const TW* __restri
                                      const int* __restrict__ positions, int n_positions) {
   constexpr int PER = 16 / (int)sizeof(TW);
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(table, ids, pos_table, positions);
   const int t = blockIdx.x;
   const int id = ids[t];
   const int at = pos_table != nullptr ? positions[t] : 0;
@@ -71,7 +71,7 @@ __global__ void embedding_pair_kernel(float* __restrict__ out, const TW* __restr
                                       const int* __restrict__ tok_pos, const int* __restrict__ last_token, int hidden,
                                       int vocab, int buckets, int mul_prev, int mul_cur, int* __restrict__ error_flag) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(table, pairs, ids, tok_slot, tok_pos, last_token);
   const int t = blockIdx.x;
   const int id = ids[t], slot = tok_slot[t];
   float* dst = out + (size_t)t * hidden;
@@ -96,7 +96,7 @@ __global__ void embedding_pair_state_kernel(int* __restrict__ last_token, const 
                                             const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
                                             int n_seqs) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(ids, cu_seqlens, seq_slot);
   const int s = blockIdx.x * blockDim.x + threadIdx.x;
   if (s >= n_seqs) return;
   const int slot = seq_slot[s], end = cu_seqlens[s + 1];

@@ -106,7 +106,7 @@ gemm_stream_kernel(TO* __restrict__ out, const __nv_bfloat16* __restrict__ x, co
 
   // The weights do not depend on the step: the first slabs are on their way while the kernel before
   // this one finishes.  X and the output do: wait for it here.
-  pdl_wait();
+  pdl_wait(x, w);
   // x with a pending norm (the product before this one left residual * norm weight and the parts of every
   // row's sum of squares): warp w adds the parts of rows w, w + 8, ... in a fixed order; the factors
   // 1 / sqrt(mean square + eps) multiply the finished sums below

@@ -38,7 +38,7 @@ struct HeadScanArgs {
   int parts, cols, tile_tokens, stage_floats;
 };
 
-enum { HS_G = 0, HS_B, HS_QK, HS_Q, HS_SCALARS };  // a token's numbers: decay, write factor, read factors
+constexpr int HS_NUMBERS = 5;  // a token's numbers: [TT] of (decay, write factor, q . k factor, read factor), [TT] of decay * key factor
 
 // One block of 128 threads (whole warps at least): one sequence, one head, `cols` value columns.  PARTS neighbouring
 // lanes hold C2 columns of the state between them, R rows each (every PARTS-th group of four rows, so that the lanes of
@@ -50,9 +50,11 @@ __global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanArgs a) {
   pdl_trigger();
   const int parts = a.parts, cols = a.cols, TT = a.tile_tokens, dim = a.dim, vdim = a.vdim;
   const int padded = parts * R;
-  // a stage: q | k, each [TT][padded]; v [TT][cols]; after the two stages the tile's numbers [HS_SCALARS][TT]
-  const int vec_floats = TT * padded;
-  float* num = tile + 2 * a.stage_floats;
+  // a stage: q | k, each [TT][padded]; v [TT][cols]; raw decays and raw betas, [TT] each (regions of whole 16 bytes); after
+  // the two stages the tile's numbers
+  const int vec_floats = TT * padded, v_floats = (TT * cols + 3) & ~3, tt_floats = (TT + 3) & ~3;
+  float4* num = reinterpret_cast<float4*>(tile + 2 * a.stage_floats);
+  float* num_seen = reinterpret_cast<float*>(num + TT);
   if (padded != dim || vdim % cols != 0)  // rows and columns beyond the head's stay zero
     for (int e = threadIdx.x; e < 2 * a.stage_floats; e += blockDim.x) tile[e] = 0.f;
   const int s = blockIdx.x, h = blockIdx.y;
@@ -85,6 +87,10 @@ __global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanArgs a) {
     for (int e = threadIdx.x; e < nt * vper; e += blockDim.x) {
       const int tt = e / vper, c = (e - tt * vper) * E;
       if (col0 + c < vdim) cp_async<B>(sv + tt * cols + c, a.v + (size_t)(t0 + tt) * a.v_stride + h * vdim + col0 + c);
+    }
+    for (int tt = threadIdx.x; tt < nt; tt += blockDim.x) {
+      if (a.decay != nullptr) cp_async<4>(sv + v_floats + tt, a.decay + (size_t)(t0 + tt) * a.decay_stride + h);
+      if (DELTA) cp_async<4>(sv + v_floats + tt_floats + tt, a.beta + (size_t)(t0 + tt) * a.beta_stride + h);
     }
     cp_async_commit();
   };
@@ -146,41 +152,58 @@ __global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanArgs a) {
     const float* sq = tile + stage * a.stage_floats;
     const float* sk = sq + vec_floats;
     const float* sv = sk + vec_floats;
+    float* sg = tile + stage * a.stage_floats + 2 * vec_floats + v_floats;
+    float* sb = sg + tt_floats;
     if (a.act == 1) activate_own(t0, stage);
+    for (int tt = threadIdx.x; tt < nt; tt += blockDim.x) {  // by the thread whose own copies brought the raw values
+      sg[tt] = a.decay != nullptr ? expf(-a_rate * softplusf_(sg[tt] + dt_bias)) : g_const;
+      sb[tt] = DELTA ? sigmoidf_(sb[tt]) : 1.0f;
+    }
     __syncthreads();
-    // a token's numbers, a warp a token
-    for (int tt = warp; tt < nt; tt += n_warps) {
-      float qk = 0.f, qq = 0.f, kk = 0.f;
-      for (int d = lane; d < padded; d += 32) {
-        const float x = sq[tt * padded + d], y = sk[tt * padded + d];
-        qk = fmaf(x, y, qk);
-        qq = fmaf(x, x, qq);
-        kk = fmaf(y, y, kk);
+    // the tokens' numbers: a warp takes four tokens at a time, whose sums run side by side
+    for (int first = 4 * warp; first < nt; first += 4 * n_warps) {
+      float qk[4] = {}, qq[4] = {}, kk[4] = {};
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int row = min(first + x, nt - 1) * padded;
+        for (int d = lane; d < padded; d += 32) {
+          const float q = sq[row + d], k = sk[row + d];
+          qk[x] = fmaf(q, k, qk[x]);
+          qq[x] = fmaf(q, q, qq[x]);
+          kk[x] = fmaf(k, k, kk[x]);
+        }
       }
-      qk = warp_sum(qk);
-      float fq = a.q_scale, fk = 1.0f;
+#pragma unroll
+      for (int x = 0; x < 4; ++x) qk[x] = warp_sum(qk[x]);
       if (a.unit_eps >= 0.f) {
-        fq = a.q_scale / sqrtf(warp_sum(qq) + a.unit_eps);
-        fk = 1.0f / sqrtf(warp_sum(kk) + a.unit_eps);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) { qq[x] = warp_sum(qq[x]); kk[x] = warp_sum(kk[x]); }
       }
-      if (lane == 0) {
-        const size_t t = (size_t)(t0 + tt);
-        float g = g_const, b = 1.0f;
-        if (a.decay != nullptr) g = expf(-a_rate * softplusf_(a.decay[t * a.decay_stride + h] + dt_bias));
-        if (DELTA) b = sigmoidf_(a.beta[t * a.beta_stride + h]);
-        num[HS_G * TT + tt] = g;
-        num[HS_B * TT + tt] = b * fk;      // plain: what v is multiplied by; delta: b times the key's factor
-        num[HS_QK * TT + tt] = qk * fq;    // what the write gives back to the read-out
-        num[HS_Q * TT + tt] = fq;
-        if (DELTA) num[HS_SCALARS * TT + tt] = g * fk;  // what S^T k (k without its factor) counts in u
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        if (lane != x || first + x >= nt) continue;
+        float fq = a.q_scale, fk = 1.0f;
+        if (a.unit_eps >= 0.f) {
+          fq = a.q_scale / sqrtf(qq[x] + a.unit_eps);
+          fk = 1.0f / sqrtf(kk[x] + a.unit_eps);
+        }
+        const float g = sg[first + x];
+        // (g, what v or its correction is multiplied by, what the write gives back to the read-out, what S^T q counts)
+        num[first + x] = make_float4(g, sb[first + x] * fk, qk[x] * fq, fq * g);
+        num_seen[first + x] = g * fk;  // what S^T k (k without its factor) counts in the correction
       }
     }
     __syncthreads();
+    float4 kn[R / 4], qn[R / 4];  // the next token's k and q are on their way while a token is worked on
+    {
+      const float4* pq = reinterpret_cast<const float4*>(sq) + part;
+      const float4* pk = reinterpret_cast<const float4*>(sk) + part;
+#pragma unroll
+      for (int i = 0; i < R / 4; ++i) { kn[i] = pk[i * parts]; qn[i] = pq[i * parts]; }
+    }
     for (int tt = 0; tt < nt; ++tt) {
-      // the lane's i-th group of four rows is 16-byte element i * parts of these
-      const float4* pq = reinterpret_cast<const float4*>(sq + tt * padded) + part;
-      const float4* pk = reinterpret_cast<const float4*>(sk + tt * padded) + part;
-      const float g = num[HS_G * TT + tt], b = num[HS_B * TT + tt], qk = num[HS_QK * TT + tt], fq = num[HS_Q * TT + tt];
+      const float4 n = num[tt];
+      const float g = n.x, b = n.y, qk = n.z, g_read = n.w, g_seen = DELTA ? num_seen[tt] : 0.f;
       float u[C2];
 #pragma unroll
       for (int c = 0; c < C2; ++c) u[c] = sv[tt * cols + jl + c];
@@ -190,9 +213,9 @@ __global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanArgs a) {
       for (int c = 0; c < C2; ++c) seen[c][0] = seen[c][1] = read[c][0] = read[c][1] = make_float2(0.f, 0.f);
 #pragma unroll
       for (int i = 0; i < R; i += 4) {
-        const float4 kq = pk[(i / 4) * parts], qq = pq[(i / 4) * parts];
-        kr[i / 2] = make_float2(kq.x, kq.y);
-        kr[i / 2 + 1] = make_float2(kq.z, kq.w);
+        kr[i / 2] = make_float2(kn[i / 4].x, kn[i / 4].y);
+        kr[i / 2 + 1] = make_float2(kn[i / 4].z, kn[i / 4].w);
+        const float4 qq = qn[i / 4];
 #pragma unroll
         for (int c = 0; c < C2; ++c) {
           if (DELTA) {
@@ -202,6 +225,14 @@ __global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanArgs a) {
           read[c][0] = __ffma2_rn(S[c][i / 2], make_float2(qq.x, qq.y), read[c][0]);
           read[c][1] = __ffma2_rn(S[c][i / 2 + 1], make_float2(qq.z, qq.w), read[c][1]);
         }
+      }
+      {
+        // the lane's i-th group of four rows is 16-byte element i * parts of these
+        const int next = min(tt + 1, nt - 1) * padded;
+        const float4* pq = reinterpret_cast<const float4*>(sq + next) + part;
+        const float4* pk = reinterpret_cast<const float4*>(sk + next) + part;
+#pragma unroll
+        for (int i = 0; i < R / 4; ++i) { kn[i] = pk[i * parts]; qn[i] = pq[i * parts]; }
       }
       float along[C2], out[C2];
 #pragma unroll
@@ -216,11 +247,10 @@ __global__ void __launch_bounds__(128) head_scan_kernel(const HeadScanArgs a) {
           out[c] += __shfl_xor_sync(0xffffffffu, out[c], o);
         }
       }
-      const float g_seen = DELTA ? num[HS_SCALARS * TT + tt] : 0.f;
 #pragma unroll
       for (int c = 0; c < C2; ++c) {
         u[c] = DELTA ? b * (u[c] - g_seen * along[c]) : b * u[c];
-        out[c] = fmaf(fq * g, out[c], qk * u[c]);
+        out[c] = fmaf(g_read, out[c], qk * u[c]);
         const float2 uu = make_float2(u[c], u[c]), gg = make_float2(g, g);
 #pragma unroll
         for (int i = 0; i < R / 2; ++i) S[c][i] = __ffma2_rn(S[c][i], gg, __fmul2_rn(kr[i], uu));
@@ -282,8 +312,8 @@ XRT_EXPORT int xrt_head_scan(float* out, const float* q, int q_stride, const flo
     per_lane >>= 1;
   while (groups > 1 && (groups / 2) * per_lane >= vdim && (groups / 2) * parts >= 32) groups >>= 1;
   const int cols = groups * per_lane, padded = parts * R;
-  auto stage_floats = [&](int tt) { return 2 * tt * padded + ((tt * cols + 3) & ~3); };
-  auto bytes = [&](int tt) { return (2 * (size_t)stage_floats(tt) + (xrt::HS_SCALARS + 1) * tt) * sizeof(float); };
+  auto stage_floats = [&](int tt) { return 2 * tt * padded + ((tt * cols + 3) & ~3) + 2 * ((tt + 3) & ~3); };
+  auto bytes = [&](int tt) { return (2 * (size_t)stage_floats(tt) + xrt::HS_NUMBERS * tt) * sizeof(float); };
   int tile_tokens = 16;
   while (tile_tokens > 1 && bytes(tile_tokens) > 46 * 1024) tile_tokens >>= 1;
   while (tile_tokens > 1 && tile_tokens / 2 >= max_new) tile_tokens >>= 1;

@@ -31,7 +31,7 @@ latent_prepare_kernel(TQ* __restrict__ q_rows, TC* __restrict__ pool, const floa
                       const int* __restrict__ block_table, int max_blocks, int n_heads, int dim, int rot, int rank,
                       int head_size, int write_cache, int interleaved) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(qd, norm_w, cos_sin, tok_slot, tok_pos, block_table);
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int slot = tok_slot[t];
   TQ* q_row = q_rows + (size_t)t * n_heads * head_size;
@@ -84,7 +84,7 @@ head_product_kernel(TO* __restrict__ out, int out_stride, int out_head, int out_
   __shared__ float xs[HP_K][HP_T + 4];
   __shared__ float ws[HP_K][HP_N + 4];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, w);
   const int t0 = blockIdx.x * HP_T, head = blockIdx.y, n0 = blockIdx.z * HP_N;
   const TX* xh = x + (size_t)head * x_head + x_off;
   const TW* wh = w + (size_t)head * n * k;
@@ -147,7 +147,7 @@ head_product_mma_kernel(__nv_bfloat16* __restrict__ out, int out_stride, int out
   __shared__ __align__(16) __nv_bfloat16 xs[BM][LD];
   __shared__ __align__(16) __nv_bfloat16 ws[BN][LD];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, w);
   const int t0 = blockIdx.x * BM, head = blockIdx.y, n0 = blockIdx.z * BN;
   const TX* xh = x + (size_t)head * x_head + x_off;
   const __nv_bfloat16* wh = w + (size_t)head * n * k;

@@ -122,7 +122,7 @@ __device__ __forceinline__ void lr_fold_tile(const float2 (*ab)[LD], int columns
 __global__ void __launch_bounds__(128)
 lr_gates_kernel(const RecurrenceArgs a, const float* __restrict__ r_raw, const float* __restrict__ i_raw) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(r_raw, i_raw);
   const int s = blockIdx.z, tile = blockIdx.y, slot = a.seq_slot[s];
   const int begin = a.cu_seqlens[s], len = a.cu_seqlens[s + 1] - begin;
   const int l0 = tile * LR_TILE, c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -170,7 +170,7 @@ lr_gates_mma_kernel(const RecurrenceArgs a, const __nv_bfloat16* __restrict__ w_
   } sh;
   __shared__ float2 half[64];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(w_r, w_i);
   const int s = blockIdx.z, tile = blockIdx.y, slot = a.seq_slot[s];
   const int begin = a.cu_seqlens[s], len = a.cu_seqlens[s + 1] - begin;
   const int l0 = tile * LR_TILE;
@@ -371,7 +371,7 @@ lr_step_kernel(__nv_bfloat16* __restrict__ out, const RecurrenceArgs a, const __
       }
     }
     __syncthreads();
-    if (!waited) { pdl_wait(); waited = true; }
+    if (!waited) { pdl_wait(w_r, w_i, tok_slot, tok_pos); waited = true; }
     // u of rows r0 .. r0 + LR_STEP_GROUP and channel c of all channels
     auto conv = [&](int r0, int c, float (&u)[LR_STEP_GROUP]) {
       float in[LR_STEP_GROUP][MOST];

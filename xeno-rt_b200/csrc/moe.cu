@@ -54,7 +54,7 @@ __global__ void moe_route_scores_kernel(int* __restrict__ ids, float* __restrict
                                         int groups, int keep, const RouteOptions opt) {
   extern __shared__ float group_best[];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(logits);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
   if (t >= n_tokens) return;
@@ -198,7 +198,7 @@ template <int PER_LANE>
 __global__ void moe_route_kernel(int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits,
                                  const float* __restrict__ bias, int n_tokens, int n_experts, int top) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(logits, bias);
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= n_tokens) return;
@@ -294,7 +294,7 @@ moe_experts_in_kernel(float* __restrict__ act, const TX* __restrict__ h, const T
                       int act_kind) {
   extern __shared__ float hs[];  // [width]
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(h, w_in, ids);
   const int t = blockIdx.x, c = blockIdx.y;
   constexpr int n_warps = MOE_WARPS, R = UNITS / MOE_WARPS, DEPTH = R >= 4 ? 4 : 8, G = R >= 2 ? R / 2 : 1;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -346,7 +346,7 @@ moe_experts_out_kernel(float* __restrict__ out, const float* __restrict__ act, c
                        int top) {
   extern __shared__ float ys[];  // [ff]
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(act, w_out, ids, weights);
   const int t = blockIdx.x, c = blockIdx.y;
   constexpr int n_warps = MOE_WARPS, R = UNITS / MOE_WARPS, DEPTH = R >= 4 ? 4 : 8;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -379,7 +379,7 @@ moe_group_kernel(int* __restrict__ offsets, int* __restrict__ pos, int* __restri
   extern __shared__ int counts[];  // [experts] counts, then [experts] cursors
   int* cursor = counts + n_experts;
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(ids);
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = 0;
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(&counts[ids[p]], 1);
@@ -405,7 +405,7 @@ template <typename TX>
 __global__ void moe_gather_kernel(TX* __restrict__ out, const TX* __restrict__ h, const int* __restrict__ row_token,
                                   int width) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(h, row_token);
   const TX* src = h + (size_t)row_token[blockIdx.x] * width;
   TX* dst = out + (size_t)blockIdx.x * width;
   for (int k = threadIdx.x; k < width; k += blockDim.x) dst[k] = src[k];
@@ -416,7 +416,7 @@ template <typename TO>
 __global__ void moe_activation_kernel(TO* __restrict__ act, const float* __restrict__ gate_up, size_t total, int ff,
                                       float limit, float alpha, float up_shift, int act_kind) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(gate_up);
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     if (act_kind == MOE_ACT_GELU) {  // gate_up holds [rows, ff]
       act[i] = from_float<TO>(gelu_erf(gate_up[i]));
@@ -433,7 +433,7 @@ __global__ void moe_activation_kernel(TO* __restrict__ act, const float* __restr
 __global__ void moe_combine_kernel(float* __restrict__ out, const float* __restrict__ y, const int* __restrict__ pos,
                                    const float* __restrict__ weights, int n_tokens, int width, int top) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(y, pos, weights);
   const int t = blockIdx.x, c = blockIdx.y;
   const float w = weights[(size_t)t * top + c];
   const float* src = y + (size_t)pos[(size_t)t * top + c] * width;

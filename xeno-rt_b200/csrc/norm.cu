@@ -53,7 +53,7 @@ rmsnorm_vec_kernel(TO* __restrict__ out, const float* __restrict__ x, const TW* 
     const int c = (threadIdx.x + i * NORM_THREADS) * 4;
     if (c < width) Vec4Of<TW>::load(w + c, wv[i]);
   }
-  pdl_wait();
+  pdl_wait(x, w, rows);
   const int r = blockIdx.x;
   const int src = rows != nullptr ? rows[r] : r;
   const float* xr = x + (size_t)src * width;
@@ -90,7 +90,7 @@ __global__ void rmsnorm_kernel(TO* __restrict__ out, const float* __restrict__ x
                                const int* __restrict__ rows, int width, float eps) {
   __shared__ float scratch[33];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, w, rows);
   const int r = blockIdx.x;
   const int src = rows != nullptr ? rows[r] : r;
   const float* xr = x + (size_t)src * width;
@@ -122,7 +122,7 @@ layernorm_vec_kernel(TO* __restrict__ out, const float* __restrict__ x, const TW
     const int c = (threadIdx.x + i * NORM_THREADS) * 4;
     if (c < width) Vec4Of<TW>::load(w + c, wv[i]);
   }
-  pdl_wait();
+  pdl_wait(x, w, rows);
   const int r = blockIdx.x;
   const int src = rows != nullptr ? rows[r] : r;
   const float* xr = x + (size_t)src * width;
@@ -170,7 +170,7 @@ __global__ void layernorm_kernel(TO* __restrict__ out, const float* __restrict__
                                  const int* __restrict__ rows, int width, float eps) {
   __shared__ float scratch[33];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, w, rows);
   const int r = blockIdx.x;
   const int src = rows != nullptr ? rows[r] : r;
   const float* xr = x + (size_t)src * width;
@@ -215,7 +215,7 @@ __global__ void layernorm_affine_kernel(TO* __restrict__ out, float* __restrict_
   extern __shared__ float row[];
   __shared__ float scratch[4][32];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, w, b, rows, w2, b2);
   const int r = blockIdx.x;
   const int src = rows != nullptr ? rows[r] : r;
   const float* xr = x + (size_t)src * width;
@@ -278,7 +278,7 @@ layernorm_affine_rows_kernel(TO* __restrict__ out, float* __restrict__ residual,
     w2v[i] = in && w2 != nullptr ? w2[c] : 0.f;
     b2v[i] = in && b2 != nullptr ? b2[c] : 0.f;
   }
-  pdl_wait();
+  pdl_wait(x, w, b, rows, w2, b2);
   const int r = blockIdx.x;
   const int src = rows != nullptr ? rows[r] : r;
   const float* xr = x + (size_t)src * width;

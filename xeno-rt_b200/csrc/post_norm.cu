@@ -35,7 +35,7 @@ __global__ void rmsnorm_add_kernel(float* __restrict__ residual, const float* __
     const int c = threadIdx.x + i * blockDim.x;
     wv[i] = c < width ? to_float(w[c]) : 0.f;
   }
-  pdl_wait();
+  pdl_wait(y, w);
   const float* p = y + (size_t)blockIdx.x * width;
   float* r = residual + (size_t)blockIdx.x * width;
   float sum = 0.f;
@@ -96,7 +96,7 @@ __global__ void rmsnorm_add_kernel(float* __restrict__ residual, const float* __
 template <typename TC>
 __global__ void cast_rows_kernel(TC* __restrict__ out, const float* __restrict__ x, size_t total) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x);
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
     out[i] = from_float<TC>(x[i]);
 }

@@ -18,7 +18,7 @@ namespace xrt {
 __global__ void rope_table_kernel(float2* __restrict__ cos_sin, const int* __restrict__ pos,
                                   const float* __restrict__ freq, float scale, int n_tokens, int half) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(pos, freq);
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n_tokens * half) return;
   const int t = i / half, p = i - t * half;
@@ -37,7 +37,7 @@ __global__ void rotation_table_kernel(float2* __restrict__ cos_sin, const int* _
                                       const float* __restrict__ freq, const float* __restrict__ freq_lo, float magnitude,
                                       int n_tokens, int half) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(pos, freq, freq_lo);
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n_tokens * half) return;
   const int t = i / half, p = i - t * half;
@@ -97,7 +97,7 @@ __global__ void qk_rope_kv_write_kernel(
     int n_heads, int n_kv_heads, int head_dim, int write_kv, int interleaved, const QueryTemp temp, const HeadExtras ex) {
   extern __shared__ float staged[];  // [warps][head_dim]
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(qkv, q_norm_w, k_norm_w, cos_sin, tok_slot, tok_pos, block_table);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
   const int head_slot = blockIdx.y * (blockDim.x >> 5) + warp;
@@ -271,7 +271,7 @@ qk_rope_kv_write_128_kernel(
     for (int j = 0; j < 4; ++j) { qn[j] = to_float(q_norm_w[4 * lane + j]); kn[j] = to_float(k_norm_w[4 * lane + j]); }
   }
   const float q_factor = temp.at(pos);
-  pdl_wait();
+  pdl_wait(qkv, q_norm_w, k_norm_w, cos_sin, tok_slot, tok_pos, block_table);
   // (cos, sin) of this lane's four pairs: dims 4 * (lane % 16) .. of the first half
   float c[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
   if (rope_half > 0 && slot >= 0) {

@@ -201,7 +201,7 @@ sample_kernel(int* __restrict__ out_ids, const float* __restrict__ logits, int v
   unsigned int* fine_hist = reinterpret_cast<unsigned int*>(dynamic);  // 4,096 bins, before the candidates are written
 
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(logits, row_slot, temperature, top_k, top_p, penalty, seen);
   const int row = blockIdx.x;
   const int slot = row_slot[row];
   if (slot < 0) { if (threadIdx.x == 0) out_ids[row] = -1; return; }

@@ -175,7 +175,7 @@ __global__ void gated_group_norm_kernel(TO* __restrict__ out, const float* __res
                                         int z_stride, const float* __restrict__ w, int width, int groups, float eps) {
   __shared__ float scratch[33];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(y, z, w);
   const int t = blockIdx.x, g = blockIdx.y;
   const int per = width / groups;
   const float* yr = y + (size_t)t * width + g * per;

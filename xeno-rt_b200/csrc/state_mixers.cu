@@ -286,7 +286,7 @@ __global__ void short_conv_kernel(float* __restrict__ out, const float* __restri
                                   const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot, int channels,
                                   int taps, int tile_tokens, int act) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, w, bias, in_bias, state, cu_seqlens, seq_slot);
   const int s = blockIdx.x;
   const int slot = seq_slot[s];
   const int begin = cu_seqlens[s], len = cu_seqlens[s + 1] - begin;
@@ -315,7 +315,7 @@ __global__ void short_conv_state_kernel(float* __restrict__ state, const float* 
                                         const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
                                         int channels, int taps) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, in_bias, cu_seqlens, seq_slot);
   const int s = blockIdx.x;
   const int slot = seq_slot[s];
   const int begin = cu_seqlens[s], len = cu_seqlens[s + 1] - begin;
@@ -348,7 +348,7 @@ __global__ void short_conv_single_kernel(float* __restrict__ out, const float* _
                                          const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot,
                                          int channels, int taps, int act) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, w, bias, in_bias, cu_seqlens, seq_slot);
   const int s = blockIdx.x;
   const int slot = seq_slot[s];
   const int begin = cu_seqlens[s], len = cu_seqlens[s + 1] - begin;
@@ -379,7 +379,7 @@ __global__ void short_conv_single_kernel(float* __restrict__ out, const float* _
 __global__ void decay_kernel(float* __restrict__ a, const float* __restrict__ bias, const float* __restrict__ a_log,
                              size_t total, int width, int dim, int mode, float tau) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(bias, a_log);
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const int c = (int)(i % width);
     const float z = a[i] + (bias != nullptr ? bias[c] : 0.f);
@@ -413,7 +413,7 @@ __global__ void removal_gates_kernel(float* __restrict__ decay, int decay_stride
                                      const float* __restrict__ k, int k_stride, int n_tokens, int n_heads, int dim,
                                      float rate, float unit_eps) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(decay_bias, removal_bias, k);
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= n_tokens * n_heads) return;
   const int t = warp / n_heads, head = warp - t * n_heads;
@@ -439,7 +439,7 @@ __global__ void head_norm_gate_kernel(TO* __restrict__ y, const float* __restric
                                       const float* __restrict__ gate, int gate_stride, int n_tokens, int n_heads,
                                       int vdim, float eps, int act, int w_per_head) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(o, w, gate);
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= n_tokens * n_heads) return;
   const int t = warp / n_heads, head = warp - t * n_heads;
@@ -454,12 +454,52 @@ __global__ void head_norm_gate_kernel(TO* __restrict__ y, const float* __restric
   for (int d = lane; d < vdim; d += 32) dst[d] = from_float<TO>((p[d] * inv) * wh[d] * activate(g[d], act));
 }
 
+// The same with a block of 256 threads a (token, head), for heads as wide as a model; PER columns a thread are asked for
+// before the sum.
+template <typename TO, int PER>
+__global__ void __launch_bounds__(256)
+wide_norm_gate_kernel(TO* __restrict__ y, const float* __restrict__ o, const float* __restrict__ w,
+                      const float* __restrict__ gate, int gate_stride, int n_heads, int vdim, float eps, int act,
+                      int w_per_head) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  const int t = blockIdx.x, head = blockIdx.y;
+  const float* wh = w + (w_per_head ? head * vdim : 0);
+  float wv[PER], ov[PER], gv[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = threadIdx.x + i * 256;
+    wv[i] = c < vdim ? wh[c] : 0.f;
+  }
+  pdl_wait(o, w, gate);
+  const float* p = o + ((size_t)t * n_heads + head) * vdim;
+  const float* g = gate + (size_t)t * gate_stride + head * vdim;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = threadIdx.x + i * 256;
+    ov[i] = c < vdim ? p[c] : 0.f;
+    gv[i] = c < vdim ? g[c] : 0.f;
+  }
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) sum = fmaf(ov[i], ov[i], sum);
+  for (int c = threadIdx.x + PER * 256; c < vdim; c += 256) sum = fmaf(p[c], p[c], sum);
+  const float inv = 1.0f / sqrtf(block_sum(sum, scratch) / (float)vdim + eps);
+  TO* dst = y + ((size_t)t * n_heads + head) * vdim;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int c = threadIdx.x + i * 256;
+    if (c < vdim) dst[c] = from_float<TO>((ov[i] * inv) * wv[i] * activate(gv[i], act));
+  }
+  for (int c = threadIdx.x + PER * 256; c < vdim; c += 256) dst[c] = from_float<TO>((p[c] * inv) * wh[c] * activate(g[c], act));
+}
+
 // x[t, c] *= act(gate[t, c]) in place.
 template <typename TX>
 __global__ void gate_mul_kernel(TX* __restrict__ x, const float* __restrict__ gate, int gate_stride, int n_tokens,
                                 int width, int act, int group) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(gate);
   const size_t total = (size_t)n_tokens * width;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const size_t t = i / width, c = i - t * width;
@@ -480,7 +520,7 @@ __global__ void rms_scale_add_kernel(float* __restrict__ residual, const float* 
     const int c = threadIdx.x + i * blockDim.x;
     wv[i] = c < width ? w[c] : 0.f;
   }
-  pdl_wait();
+  pdl_wait(y, w);
   const float* p = y + (size_t)blockIdx.x * width;
   float* r = residual + (size_t)blockIdx.x * width;
   float sum = 0.f;
@@ -508,7 +548,7 @@ template <typename TO>
 __global__ void concat_cast_kernel(TO* __restrict__ out, const float* __restrict__ a, const float* __restrict__ b,
                                    int n_tokens, int width) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(a, b);
   const size_t total = (size_t)n_tokens * 2 * width;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const size_t t = i / (2 * width), c = i - t * 2 * width;
@@ -521,7 +561,7 @@ template <typename TO>
 __global__ void act_cast_kernel(TO* __restrict__ out, const float* __restrict__ x, int x_stride, int n_tokens, int width,
                                 int act) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x);
   const size_t total = (size_t)n_tokens * width;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const size_t t = i / width, c = i - t * width;
@@ -533,7 +573,7 @@ __global__ void act_cast_kernel(TO* __restrict__ out, const float* __restrict__ 
 __global__ void add_scaled_parts_kernel(float* __restrict__ residual, const float* __restrict__ parts,
                                         const float* __restrict__ scales, size_t total, int n_parts) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(parts, scales);
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     float sum = 0.f;
     for (int p = 0; p < n_parts; ++p) sum = fmaf(parts[(size_t)p * total + i], scales[p], sum);
@@ -691,6 +731,17 @@ XRT_EXPORT int xrt_head_norm_gate(void* y, const float* o, const float* w, const
                                   int w_per_head, cudaStream_t stream) {
   if (n_tokens < 0 || n_heads <= 0 || vdim <= 0 || gate_stride < n_heads * vdim) return XRT_ERR_ARGUMENT;
   if (n_tokens == 0) return XRT_OK;
+  if (vdim > 512 && n_heads <= 65535) {
+    XRT_DISPATCH_DTYPE(out_dtype, TO, {
+      if (vdim <= 1024)
+        xrt::launch_kernel(xrt::wide_norm_gate_kernel<TO, 4>, dim3(n_tokens, n_heads), dim3(256), 0, stream, (TO*)y, o, w, gate,
+                           gate_stride, n_heads, vdim, eps, act, w_per_head);
+      else
+        xrt::launch_kernel(xrt::wide_norm_gate_kernel<TO, 8>, dim3(n_tokens, n_heads), dim3(256), 0, stream, (TO*)y, o, w, gate,
+                           gate_stride, n_heads, vdim, eps, act, w_per_head);
+    });
+    return xrt::launch_status();
+  }
   const size_t warps = (size_t)n_tokens * n_heads;
   XRT_DISPATCH_DTYPE(out_dtype, TO, {
     xrt::launch_kernel(xrt::head_norm_gate_kernel<TO>, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0, stream, (TO*)y, o,

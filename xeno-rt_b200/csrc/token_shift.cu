@@ -38,7 +38,7 @@ __global__ void rmsnorm_shift_kernel(TO* __restrict__ out, const float* __restri
   const int pos = tok_pos[t];
   const bool inside = t > 0 && tok_slot[t - 1] == slot;  // the token before is a row of this step
   const bool last = t + 1 >= n_tokens || tok_slot[t + 1] != slot;
-  pdl_wait();
+  pdl_wait(x, w, shift, tok_slot, tok_pos);
   TO* dst = out + (size_t)t * width;
   if (slot < 0) {  // a padding row
     for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = from_float<TO>(0.f);
@@ -80,7 +80,7 @@ __global__ void rmsnorm_shift_state_kernel(float* __restrict__ state, const floa
                                            const int* __restrict__ seq_slot, int width, float eps) {
   __shared__ float scratch[33];
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(x, w, cu_seqlens, seq_slot);
   const int s = blockIdx.x;
   const int slot = seq_slot[s];
   const int begin = cu_seqlens[s], end = cu_seqlens[s + 1];
@@ -105,7 +105,7 @@ __global__ void rmsnorm_shift_state_kernel(float* __restrict__ state, const floa
 template <typename TW>
 __global__ void add_row_kernel(float* __restrict__ x, const TW* __restrict__ row, size_t total, int width) {
   pdl_trigger();
-  pdl_wait();
+  pdl_wait(row);
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
     x[i] += to_float(row[i % width]);
 }

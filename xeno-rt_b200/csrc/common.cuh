@@ -282,6 +282,20 @@ inline void launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_
   cudaLaunchKernelEx(&config, kernel, static_cast<KArgs>(args)...);
 }
 
+// A launch that waits for the kernel before it as a whole: for few blocks that run long.  Launched early, such blocks
+// would be placed where the kernel before leaves room first, several on one multiprocessor while others stay empty
+// (measured: twice the time for the scans of a prompt).
+template <typename... KArgs, typename... Args>
+inline void launch_kernel_alone(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                                Args... args) {
+  cudaLaunchConfig_t config = {};
+  config.gridDim = grid;
+  config.blockDim = block;
+  config.dynamicSmemBytes = smem;
+  config.stream = stream;
+  cudaLaunchKernelEx(&config, kernel, static_cast<KArgs>(args)...);
+}
+
 // The same launch with a range of global memory that the kernel reads once (a weight): its lines
 // are marked as streaming in the L2 (an access-policy window of the launch), so they are the first to
 // leave and what the step reads again stays.  For kernels whose copies cannot carry a cache hint

@@ -32,7 +32,7 @@ _SIGNATURES = {
     "xrt_swiglu": [_P, _P, _I, _I, _I, _I, _I, _P, _P],
     "xrt_rotation_table": [_P, _P, _P, _P, _F, _I, _I, _P],
     "xrt_state_scan": [_P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
-    "xrt_head_scan": [_P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _P],
+    "xrt_head_scan": [_P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _P, _P],
     "xrt_stream_add": [_P, _P, ctypes.c_longlong, _I, _P, _P, _P, _P, _F, _F, _P, _P, _F, _I, _I, _I, _I, _P],
     "xrt_removal_gates": [_P, _I, _P, _P, _I, _P, _P, _I, _P, _I, _I, _I, _I, _F, _F, _P],
     "xrt_rmsnorm_shift": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _P],
@@ -954,7 +954,8 @@ def head_scan(out, q, k, v, state, cu_seqlens, seq_slot, n_heads: int, n_qk_head
     raw value a token and head.  ``silu``: q, k and v pass silu first; ``unit_eps``: q and k are then divided by
     sqrt(sum(x^2) + unit_eps) a head.  q, k [T, n_qk_heads * dim], v [T, n_heads * vdim], rows may be slices of wider
     rows, all float32; ``state`` float32 [slots, n_heads, vdim, dim] is read and left as the sequences' last state.
-    ``max_new`` (0: not known): the most tokens a sequence brings."""
+    ``max_new`` (0: not known): the most tokens a sequence brings; portions of several tokens without ``silu`` run four
+    tokens at a time."""
     n = out.shape[0]
     if out.shape != (n, n_heads * vdim) or out.dtype != torch.float32 or not out.is_contiguous():
         raise KernelError("head_scan: out must be float32 [T, heads * vdim]")
@@ -975,11 +976,15 @@ def head_scan(out, q, k, v, state, cu_seqlens, seq_slot, n_heads: int, n_qk_head
     vp, vs = _columns(v, "v", n_heads * vdim)
     dp, ds = _columns(decay_raw, "decay_raw", n_heads) if decay_raw is not None else (0, 0)
     bp, bs = _columns(beta, "beta", n_heads) if beta is not None else (0, 0)
+    terms = None
+    if max_new > 1 and not silu and dim <= 512:  # portions run four tokens at a time from terms made first
+        terms = torch.empty((n // 4 + n_seqs + 1) * n_heads * 32, dtype=torch.float32, device=out.device)
+        add_launches(1)
     _check(_kernels().xrt_head_scan(
         _ptr(out, "out"), qp, qs, kp, ks, vp, vs, dp, ds, _ptr(decay, "decay", torch.float32),
         _ptr(a_log, "a_log", torch.float32), _ptr(dt_bias, "dt_bias", torch.float32), bp, bs, _ptr(state, "state"),
         _ptr(cu_seqlens, "cu_seqlens", torch.int32), _ptr(seq_slot, "seq_slot", torch.int32), n_seqs, n_heads, n_qk_heads,
-        dim, vdim, float(q_scale), -1.0 if unit_eps is None else float(unit_eps), 1 if silu else 0, int(max_new), _stream()),
+        dim, vdim, float(q_scale), -1.0 if unit_eps is None else float(unit_eps), 1 if silu else 0, int(max_new), _ptr(terms, "terms"), _stream()),
         "head_scan")
 
 

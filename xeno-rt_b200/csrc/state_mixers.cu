@@ -507,6 +507,49 @@ __global__ void gate_mul_kernel(TX* __restrict__ x, const float* __restrict__ ga
   }
 }
 
+// The two above for widths and strides of whole fours: blocks of a token's columns, four a thread, no divisions.
+template <typename T>
+__device__ __forceinline__ void store_four(T* dst, const float (&v)[4]) {
+  alignas(16) T o[4];
+#pragma unroll
+  for (int x = 0; x < 4; ++x) o[x] = from_float<T>(v[x]);
+  if (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(o);
+  else *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(o);
+}
+
+template <typename TX>
+__global__ void __launch_bounds__(256) gate_mul_rows_kernel(TX* __restrict__ x, const float* __restrict__ gate,
+                                                            int gate_stride, int width, int act, int group) {
+  pdl_trigger();
+  pdl_wait(gate);
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  if (c >= width) return;
+  TX* p = x + (size_t)blockIdx.x * width + c;
+  const float* g = gate + (size_t)blockIdx.x * gate_stride;
+  float f[4], v[4];
+  if (group == 1) {
+    const float4 t = *reinterpret_cast<const float4*>(g + c);
+    f[0] = t.x; f[1] = t.y; f[2] = t.z; f[3] = t.w;
+  } else {  // (group is a multiple of four: one gate for all)
+    f[0] = f[1] = f[2] = f[3] = g[c / group];
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) v[i] = to_float(p[i]) * activate(f[i], act);
+  store_four(p, v);
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(256) act_cast_rows_kernel(TO* __restrict__ out, const float* __restrict__ x, int x_stride,
+                                                            int width, int act) {
+  pdl_trigger();
+  pdl_wait(x);
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  if (c >= width) return;
+  const float4 t = *reinterpret_cast<const float4*>(x + (size_t)blockIdx.x * x_stride + c);
+  const float v[4] = {activate(t.x, act), activate(t.y, act), activate(t.z, act), activate(t.w, act)};
+  store_four(out + (size_t)blockIdx.x * width + c, v);
+}
+
 // residual[t] += factor * y[t] / sqrt(mean(y[t]^2) + eps) * w; one block a row.  The row, the weight and the
 // residual are all asked for before the sum (a few rows a step: the time is load latency).
 template <int PER>
@@ -648,7 +691,11 @@ XRT_EXPORT int xrt_state_scan(float* out, const float* q, int q_stride, const fl
                      cu_seqlens, seq_slot, n_heads, n_heads / n_qk_heads, dim, vdim, q_scale, parts, cols, tile_tokens,
                      stage_floats(tile_tokens)};
   const dim3 grid(n_seqs, n_heads, (vdim + cols - 1) / cols), block(parts * groups);
-#define XRT_SCAN(RR, CC, DD, VV) xrt::launch_kernel(xrt::state_scan_kernel<RR, CC, DD, VV>, grid, block, smem, stream, a)
+#define XRT_SCAN(RR, CC, DD, VV)                                                                                  \
+  do {                                                                                                                \
+    if (max_new > 1) xrt::launch_kernel_alone(xrt::state_scan_kernel<RR, CC, DD, VV>, grid, block, smem, stream, a);  \
+    else xrt::launch_kernel(xrt::state_scan_kernel<RR, CC, DD, VV>, grid, block, smem, stream, a);                    \
+  } while (0)
 #define XRT_SCAN_R(RR, CC)                                     \
   do {                                                         \
     if (mode == 2 && vec) XRT_SCAN(RR, CC, 2, true);           \
@@ -754,6 +801,14 @@ XRT_EXPORT int xrt_gate_mul(void* x, const float* gate, int gate_stride, int n_t
                             int group, cudaStream_t stream) {
   if (n_tokens < 0 || width <= 0 || group <= 0 || width % group || gate_stride < width / group) return XRT_ERR_ARGUMENT;
   if (n_tokens == 0) return XRT_OK;
+  if (width % 4 == 0 && gate_stride % 4 == 0 && (group == 1 || group % 4 == 0) && width / 4 <= 65535 * 256 &&
+      (((uintptr_t)x | (uintptr_t)gate) & 15) == 0) {
+    XRT_DISPATCH_DTYPE(dtype, TX, {
+      xrt::launch_kernel(xrt::gate_mul_rows_kernel<TX>, dim3(n_tokens, (width / 4 + 255) / 256), dim3(256), 0, stream, (TX*)x,
+                         gate, gate_stride, width, act, group);
+    });
+    return xrt::launch_status();
+  }
   XRT_DISPATCH_DTYPE(dtype, TX, {
     xrt::launch_kernel(xrt::gate_mul_kernel<TX>, dim3(xrt::grid_for((size_t)n_tokens * width, 256)), dim3(256), 0, stream,
                        (TX*)x, gate, gate_stride, n_tokens, width, act, group);
@@ -790,6 +845,13 @@ XRT_EXPORT int xrt_act_cast(void* out, const float* x, int x_stride, int n_token
                             cudaStream_t stream) {
   if (n_tokens < 0 || width <= 0 || x_stride < width) return XRT_ERR_ARGUMENT;
   if (n_tokens == 0) return XRT_OK;
+  if (width % 4 == 0 && x_stride % 4 == 0 && width / 4 <= 65535 * 256 && (((uintptr_t)out | (uintptr_t)x) & 15) == 0) {
+    XRT_DISPATCH_DTYPE(out_dtype, TO, {
+      xrt::launch_kernel(xrt::act_cast_rows_kernel<TO>, dim3(n_tokens, (width / 4 + 255) / 256), dim3(256), 0, stream, (TO*)out,
+                         x, x_stride, width, act);
+    });
+    return xrt::launch_status();
+  }
   XRT_DISPATCH_DTYPE(out_dtype, TO, {
     xrt::launch_kernel(xrt::act_cast_kernel<TO>, dim3(xrt::grid_for((size_t)n_tokens * width, 256)), dim3(256), 0, stream,
                        (TO*)out, x, x_stride, n_tokens, width, act);

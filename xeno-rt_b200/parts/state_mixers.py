@@ -265,8 +265,12 @@ class ConstantDecayLinearAttention(_StateMixer):
         n = h.shape[0]
         p = linear(h, self.w_in, out_dtype=torch.float32)   # q | k | v | g
         o = self._rows(ctx)((n, nh * vd), dtype=torch.float32, device=h.device)
-        ops.head_scan(o, p, p[:, nh * kd:], p[:, 2 * nh * kd:], store.state, ctx.cu_seqlens, ctx.seq_slot, nh, nh, kd, vd,
-                      decay=self.decay, silu=True, max_new=ctx.max_new)
+        qkv, single = p, ctx.max_new == 1  # (the scan of single tokens takes silu along; in portions it would do so many times)
+        if not single:
+            qkv = torch.empty((n, 2 * nh * kd + nh * vd), dtype=torch.float32, device=h.device)
+            ops.act_cast(qkv, p[:, :2 * nh * kd + nh * vd], "silu")
+        ops.head_scan(o, qkv, qkv[:, nh * kd:], qkv[:, 2 * nh * kd:], store.state, ctx.cu_seqlens, ctx.seq_slot, nh, nh, kd, vd,
+                      decay=self.decay, silu=single, max_new=ctx.max_new)
         y = torch.empty((n, nh * vd), dtype=self.act_dtype, device=h.device)
         ops.head_norm_gate(y, o, self.norm, p[:, 2 * nh * kd + nh * vd:], 1, nh * vd, self.eps, "sigmoid")
         return y

@@ -229,9 +229,11 @@ XRT_EXPORT int xrt_ssd_scan(float* out, const float* x, int x_stride, const floa
                    (((uintptr_t)x | (uintptr_t)b | (uintptr_t)c) & 15) == 0;
   dim3 grid(n_seqs, n_heads, (vdim + a.cols - 1) / a.cols);
 #define XRT_SSD(R)                                                                                              \
-  do {                                                                                                          \
-    if (vec) xrt::launch_kernel(xrt::ssd_scan_kernel<R, true>, grid, dim3(threads), smem, stream, a);          \
-    else xrt::launch_kernel(xrt::ssd_scan_kernel<R, false>, grid, dim3(threads), smem, stream, a);             \
+  do {                                                                                                                 \
+    if (max_new > 1 && vec) xrt::launch_kernel_alone(xrt::ssd_scan_kernel<R, true>, grid, dim3(threads), smem, stream, a); \
+    else if (max_new > 1) xrt::launch_kernel_alone(xrt::ssd_scan_kernel<R, false>, grid, dim3(threads), smem, stream, a);  \
+    else if (vec) xrt::launch_kernel(xrt::ssd_scan_kernel<R, true>, grid, dim3(threads), smem, stream, a);               \
+    else xrt::launch_kernel(xrt::ssd_scan_kernel<R, false>, grid, dim3(threads), smem, stream, a);                       \
   } while (0)
   if (r == 1) XRT_SSD(1);
   else if (r == 2) XRT_SSD(2);
